@@ -11,6 +11,9 @@
 //                        s = sum_j a[j] X[j, t, :] is written as the stream and the next norm reads s.
 //   depth_average:       s[r, :] = sum_j a[j] X[j, row(r), :], the stream itself and/or
 //                        its RMS norm in the activation dtype; row(r) = rows[r] or r.
+//   postnorm_add:        v = s0 y0[t, :] (+ s1 y1[t, :]);  x[t, :] += c v / sqrt(mean(v^2) + eps) * w, in place,
+//                        and the new x in the activation dtype beside it (what the next sublayer reads)
+//   activation_rows:     the stream in the activation dtype;   scaled_sum2: s0 a + s1 b
 // One block per row; the order of a row's additions depends on H and the block
 // size only.
 #include "common.cuh"
@@ -142,6 +145,138 @@ RLLM_EXPORT int rllm_depth_average(const float* hist, long long level_stride, in
   } while (0)
   RLLM_DISPATCH_DTYPE(act_dtype, TA_, RLLM_DISPATCH_DTYPE(w_dtype, TW_, GLUE_LAUNCH(TA_, TW_)));
 #undef GLUE_LAUNCH
+  RLLM_LAUNCH_CHECK();
+  return 0;
+}
+
+// A thread keeps its values of the row between the two passes: PN_KEEP groups of V neighbouring elements (the
+// rest of very wide rows is read again).
+#define PN_KEEP 4
+template <typename T, int V> __device__ __forceinline__ void pn_load(const T* p, float (&o)[V]) {
+  if (V == 1) { o[0] = to_f32(p[0]); return; }
+  struct alignas(V * sizeof(T)) A { T v[V]; };
+  const A a = *(const A*)p;
+#pragma unroll
+  for (int i = 0; i < V; ++i) o[i] = to_f32(a.v[i]);
+}
+template <typename T, int V> __device__ __forceinline__ void pn_store(T* p, const float (&o)[V]) {
+  if (V == 1) { p[0] = from_f32<T>(o[0]); return; }
+  struct alignas(V * sizeof(T)) A { T v[V]; };
+  A a;
+#pragma unroll
+  for (int i = 0; i < V; ++i) a.v[i] = from_f32<T>(o[i]);
+  *(A*)p = a;
+}
+
+template <typename TA, typename TW, int V>
+__global__ void __launch_bounds__(GLUE_THREADS)
+postnorm_add_kernel(float* x, const TA* y0, const TA* y1, float s0, float s1, const TW* w, float eps, float mult,
+                    TA* x_act, int H) {
+  pdl_wait();
+  pdl_launch();
+  __shared__ float red[32];
+  const size_t base = (size_t)blockIdx.x * H;
+  const int groups = H / V;
+  float keep[PN_KEEP][V];
+  auto value = [&](int g, float (&o)[V]) {
+    pn_load<TA, V>(y0 + base + (size_t)g * V, o);
+#pragma unroll
+    for (int i = 0; i < V; ++i) o[i] *= s0;
+    if (y1) {
+      float b[V];
+      pn_load<TA, V>(y1 + base + (size_t)g * V, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i) o[i] = fmaf(s1, b[i], o[i]);
+    }
+  };
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < PN_KEEP; ++u) {
+    const int g = threadIdx.x + u * blockDim.x;
+    if (g < groups) {
+      value(g, keep[u]);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss = fmaf(keep[u][i], keep[u][i], ss);
+    }
+  }
+  for (int g = threadIdx.x + PN_KEEP * blockDim.x; g < groups; g += blockDim.x) {
+    float o[V];
+    value(g, o);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss = fmaf(o[i], o[i], ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  auto finish = [&](int g, const float (&o)[V]) {
+    float h[V], wv[V];
+    pn_load<float, V>(x + base + (size_t)g * V, h);
+    pn_load<TW, V>(w + (size_t)g * V, wv);
+#pragma unroll
+    for (int i = 0; i < V; ++i) h[i] += mult * (o[i] * inv * wv[i]);
+    pn_store<float, V>(x + base + (size_t)g * V, h);
+    if (x_act) pn_store<TA, V>(x_act + base + (size_t)g * V, h);
+  };
+#pragma unroll
+  for (int u = 0; u < PN_KEEP; ++u) {
+    const int g = threadIdx.x + u * blockDim.x;
+    if (g < groups) finish(g, keep[u]);
+  }
+  for (int g = threadIdx.x + PN_KEEP * blockDim.x; g < groups; g += blockDim.x) {
+    float o[V];
+    value(g, o);
+    finish(g, o);
+  }
+}
+
+static inline int pn_threads(int groups) {
+  int n = (groups + 31) / 32 * 32;
+  return n < 32 ? 32 : (n > GLUE_THREADS ? GLUE_THREADS : n);
+}
+
+// y1 may be null (then s1 is not read); x_act may be null
+RLLM_EXPORT int rllm_postnorm_add(float* x, const void* y0, const void* y1, float s0, float s1, const void* w, float eps,
+                                  float mult, void* x_act, int T, int H, int act_dtype, int w_dtype,
+                                  cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || !x || !y0 || !w) return RLLM_E_BADARG;
+  const bool wide = H % 4 == 0 && (((uintptr_t)x | (uintptr_t)y0 | (uintptr_t)y1 | (uintptr_t)w | (uintptr_t)x_act) & 15) == 0;
+#define PN_GO(TA, TW, V)                                                                                          \
+  rllm_launch_pdl(postnorm_add_kernel<TA, TW, V>, dim3(T), dim3(pn_threads(H / V)), (size_t)0, stream, x,         \
+                  (const TA*)y0, (const TA*)y1, s0, s1, (const TW*)w, eps, mult, (TA*)x_act, H)
+  RLLM_DISPATCH_DTYPE(act_dtype, TA_, RLLM_DISPATCH_DTYPE(w_dtype, TW_, {
+    if (wide) PN_GO(TA_, TW_, 4); else PN_GO(TA_, TW_, 1);
+  }));
+#undef PN_GO
+  RLLM_LAUNCH_CHECK();
+  return 0;
+}
+
+__global__ void __launch_bounds__(256) activation_rows_kernel(const float* x, bf16* out, long long n) {
+  pdl_wait();
+  pdl_launch();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i < n) out[i] = from_f32<bf16>(x[i]);
+}
+RLLM_EXPORT int rllm_activation_rows(const float* x, void* out, long long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  rllm_launch_pdl(activation_rows_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), (size_t)0, stream, x, (bf16*)out, n);
+  RLLM_LAUNCH_CHECK();
+  return 0;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256) scaled_sum2_kernel(const T* a, const T* b, float sa, float sb, T* out, long long n) {
+  pdl_wait();
+  pdl_launch();
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i < n) out[i] = from_f32<T>(fmaf(sb, to_f32(b[i]), sa * to_f32(a[i])));
+}
+RLLM_EXPORT int rllm_scaled_sum2(const void* a, const void* b, float sa, float sb, void* out, int dtype, long long n,
+                                 cudaStream_t stream) {
+  if (n <= 0) return 0;
+  RLLM_DISPATCH_DTYPE(dtype, TT,
+    (rllm_launch_pdl(scaled_sum2_kernel<TT>, dim3((unsigned)((n + 255) / 256)), dim3(256), (size_t)0, stream, (const TT*)a,
+                     (const TT*)b, sa, sb, (TT*)out, n)));
   RLLM_LAUNCH_CHECK();
   return 0;
 }

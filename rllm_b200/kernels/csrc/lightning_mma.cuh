@@ -11,7 +11,13 @@
 // float32.  Every operand lies in shared memory as it lies in global memory (tokens by channels, the state
 // [d][dv]); where a product sums over the rows of such an array (V, S_0, K * w), its fragments come from
 // ldmatrix with .trans.
+//
+// The same passes serve the recurrence with step sizes (STEPS true, see lightning_walk.cuh): with L_t the sum of
+// the logarithms of the chunk's decays up to token t, w_j = exp(L_(n-1) - L_j) dt_j, D[t, j] = exp(L_t - L_j) dt_j
+// and the start state's row factor is exp(L_t); q and k are a group's rows, nothing is activated, and d_h v_t is
+// added.  Heads smaller than the built sizes D x DV are then filled up with zeros in shared memory.
 #pragma once
+#include "lightning_walk.cuh"
 #include "tile_gemm_mma.cuh"
 
 #define LTC_CHUNK 64
@@ -25,7 +31,25 @@ template <int D, int DVB> struct LtcSmem2 {
 };
 template <int D, int DV> struct LtcSplit { static constexpr int N = (D > 64 && DV > 64) ? 2 : 1; };
 
-__device__ __forceinline__ float ltc_silu(float v) { return v / (1.0f + expf(-v)); }
+// STEPS: the chunk's running sums of log2 decays and its step sizes, made by the first warp (two tokens a lane)
+struct LtcFactors { float L[LTC_CHUNK], dt[LTC_CHUNK]; };
+__device__ __forceinline__ void ltc_factors(LtcFactors& f, const LtSteps& p, int t0, int n, int h, int heads) {
+  if (threadIdx.x >= 32) return;
+  const int lane = threadIdx.x;
+  const float rate = expf(p.a_log[h]) * 1.4426950408889634f;
+  const float d0 = 2 * lane < n ? lt_step(p, t0 + 2 * lane, h, heads) : 0.f;
+  const float d1 = 2 * lane + 1 < n ? lt_step(p, t0 + 2 * lane + 1, h, heads) : 0.f;
+  float run = d0 + d1;                             // inclusive sums over the lanes
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const float up = __shfl_up_sync(0xffffffffu, run, o);
+    if (lane >= o) run += up;
+  }
+  f.L[2 * lane] = -rate * (run - d1);
+  f.L[2 * lane + 1] = -rate * run;
+  f.dt[2 * lane] = d0;
+  f.dt[2 * lane + 1] = d1;
+}
 __device__ __forceinline__ uint32_t ltc_pack(bf16 a, bf16 b) {
   __nv_bfloat162 p;
   p.x = a;
@@ -68,16 +92,18 @@ __device__ __forceinline__ void ltc_b_t(uint32_t (&b)[4], const bf16* base, int 
 
 // Four consecutive projections of a token's row, activated (zeros behind the chunk's n tokens).  `wide`: the
 // rows are 8-byte aligned and one load fetches the four.
-__device__ __forceinline__ void ltc_fetch4(const bf16* src, bool on, bool wide, float (&o)[4]) {
-  if (!on) {
+// (`left`: how many of the four exist; the rest are zeros)
+template <bool STEPS>
+__device__ __forceinline__ void ltc_fetch4(const bf16* src, bool on, bool wide, int left, float (&o)[4]) {
+  if (!on || left <= 0) {
     o[0] = o[1] = o[2] = o[3] = 0.f;
-  } else if (wide) {
+  } else if (wide && left >= 4) {
     const uint2 raw = *(const uint2*)src;
     const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&raw.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&raw.y);
-    o[0] = ltc_silu(a.x); o[1] = ltc_silu(a.y); o[2] = ltc_silu(b.x); o[3] = ltc_silu(b.y);
+    o[0] = lt_act<STEPS>(a.x); o[1] = lt_act<STEPS>(a.y); o[2] = lt_act<STEPS>(b.x); o[3] = lt_act<STEPS>(b.y);
   } else {
 #pragma unroll
-    for (int x = 0; x < 4; ++x) o[x] = ltc_silu(__bfloat162float(src[x]));
+    for (int x = 0; x < 4; ++x) o[x] = x < left ? lt_act<STEPS>(__bfloat162float(src[x])) : 0.f;
   }
 }
 __device__ __forceinline__ void ltc_store4(bf16* dst, const float (&o)[4]) {
@@ -87,25 +113,37 @@ __device__ __forceinline__ void ltc_store4(bf16* dst, const float (&o)[4]) {
   *(uint2*)dst = t;
 }
 
+// two neighbouring values of row i of an array [rows][cols], as far as they exist
+__device__ __forceinline__ void ltc_put2(float* base, int i, int c, int rows, int cols, float x, float y) {
+  if (i >= rows || c >= cols) return;
+  float* p = base + (size_t)i * cols + c;
+  if ((cols & 1) == 0) { *(float2*)p = make_float2(x, y); return; }
+  p[0] = x;
+  if (c + 1 < cols) p[1] = y;
+}
+
 // a chunk's rows of one projection into shared memory [token][W + 8], activated and rounded
-// (W columns from column `col0` of the head's HW)
-template <int W, int HW>
+// (W columns from column `col0` of the head's hw)
+template <int W, bool STEPS>
 __device__ __forceinline__ void ltc_stage_rows(bf16 (*dst)[W + 8], const bf16* src, int stride, int t0, int n, int h,
-                                               int col0, bool wide) {
+                                               int hw, int col0, bool wide) {
 #pragma unroll
   for (int e0 = 0; e0 < LTC_CHUNK * W; e0 += LTC_THREADS * 4) {
     const int e = e0 + threadIdx.x * 4;
     const int j = e / W, c = e - j * W;
     float o[4];
-    ltc_fetch4(src + (size_t)(t0 + j) * stride + (size_t)h * HW + col0 + c, j < n, wide, o);
+    ltc_fetch4<STEPS>(src + (size_t)(t0 + j) * stride + (size_t)h * hw + col0 + c, j < n, wide, hw - col0 - c, o);
     ltc_store4(&dst[j][c], o);
   }
 }
 
-template <int D, int DV>
+// (d, dv: the head's sizes; without STEPS they are D and DV)
+template <int D, int DV, bool STEPS>
 __global__ void __launch_bounds__(LTC_THREADS)
-lightning_mma_pass1_kernel(const bf16* k, const bf16* v, int stride, int wide, const float* decay, float* work,
-                           const int* q_start, int max_chunks, int heads) {
+lightning_mma_pass1_kernel(const bf16* k, const bf16* v, int stride, int wide, const float* decay, LtSteps steps,
+                           float* work, const int* q_start, int max_chunks, int heads, int d_, int dv_) {
+  __shared__ LtcFactors fac;
+  const int d = STEPS ? d_ : D, dv = STEPS ? dv_ : DV;
   extern __shared__ __align__(16) unsigned char ltc_raw[];
   LtcSmem1<D, DV>& sm = *reinterpret_cast<LtcSmem1<D, DV>*>(ltc_raw);
   pdl_wait();
@@ -114,14 +152,21 @@ lightning_mma_pass1_kernel(const bf16* k, const bf16* v, int stride, int wide, c
   const int t0 = q_start[s] + chunk * LTC_CHUNK;
   const int n = min(LTC_CHUNK, q_start[s + 1] - t0);
   if (n <= 0) return;
-  const float l2 = log2f(decay[h]);
+  const float l2 = STEPS ? 0.f : log2f(decay[h]);
+  const int hk = STEPS ? h / steps.per : h;
+  if (STEPS) {
+    ltc_factors(fac, steps, t0, n, h, heads);
+    __syncthreads();
+    if (threadIdx.x == 0) steps.chunk_dt[(size_t)blockIdx.y * heads + h] = -fac.L[n - 1] / (expf(steps.a_log[h]) * 1.4426950408889634f);
+  }
 #pragma unroll
   for (int e0 = 0; e0 < LTC_CHUNK * D; e0 += LTC_THREADS * 4) {
     const int e = e0 + threadIdx.x * 4;
     const int j = e / D, i = e - j * D;
     float o[4], hi[4], lo[4];
-    ltc_fetch4(k + (size_t)(t0 + j) * stride + (size_t)h * D + i, j < n, wide != 0, o);
-    const float w = (j < n) ? ltc_pow(l2, n - 1 - j) : 0.f;
+    ltc_fetch4<STEPS>(k + (size_t)(t0 + j) * stride + (size_t)hk * d + i, j < n, wide != 0, d - i, o);
+    float w = 0.f;
+    if (j < n) w = STEPS ? exp2f(fac.L[n - 1] - fac.L[j]) * fac.dt[j] : ltc_pow(l2, n - 1 - j);
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
       const float kw = __bfloat162float(__float2bfloat16_rn(o[x])) * w;      // the rounded key, weighted
@@ -131,7 +176,7 @@ lightning_mma_pass1_kernel(const bf16* k, const bf16* v, int stride, int wide, c
     ltc_store4(&sm.kh[j][i], hi);
     ltc_store4(&sm.kl[j][i], lo);
   }
-  ltc_stage_rows<DV, DV>(sm.v, v, stride, t0, n, h, 0, wide != 0);
+  ltc_stage_rows<DV, STEPS>(sm.v, v, stride, t0, n, h, dv, 0, wide != 0);
   __syncthreads();
   // a warp owns DV / 4 value columns and half of the d rows
   constexpr int MT = D / 32, NT = DV / 32;
@@ -163,22 +208,25 @@ lightning_mma_pass1_kernel(const bf16* k, const bf16* v, int stride, int wide, c
       }
     }
   }
-  float* z = work + ((size_t)blockIdx.y * heads + h) * D * DV;
+  float* z = work + ((size_t)blockIdx.y * heads + h) * d * dv;
   const int g = lane >> 2, tq = lane & 3;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
-      const int c = c0 + nt * 8 + 2 * tq;
-      *(float2*)(z + (size_t)(m0 + mt * 16 + g) * DV + c) = make_float2(acc[mt][nt][0], acc[mt][nt][1]);
-      *(float2*)(z + (size_t)(m0 + mt * 16 + g + 8) * DV + c) = make_float2(acc[mt][nt][2], acc[mt][nt][3]);
+      const int c = c0 + nt * 8 + 2 * tq, i = m0 + mt * 16 + g;
+      ltc_put2(z, i, c, d, dv, acc[mt][nt][0], acc[mt][nt][1]);
+      ltc_put2(z, i + 8, c, d, dv, acc[mt][nt][2], acc[mt][nt][3]);
     }
 }
 
-template <int D, int DV>
+template <int D, int DV, bool STEPS>
 __global__ void __launch_bounds__(LTC_THREADS)
 lightning_mma_pass2_kernel(const bf16* q, const bf16* k, const bf16* v, int stride, int wide, const float* decay,
-                           const float* work, const int* q_start, int max_chunks, float* out, int heads) {
+                           LtSteps steps, const float* work, const int* q_start, int max_chunks, float* out, int heads,
+                           int d_, int dv_) {
+  __shared__ LtcFactors fac;
+  const int d = STEPS ? d_ : D, dv = STEPS ? dv_ : DV;
   constexpr int DVB = DV / LtcSplit<D, DV>::N;
   extern __shared__ __align__(16) unsigned char ltc_raw[];
   LtcSmem2<D, DVB>& sm = *reinterpret_cast<LtcSmem2<D, DVB>*>(ltc_raw);
@@ -189,17 +237,26 @@ lightning_mma_pass2_kernel(const bf16* q, const bf16* k, const bf16* v, int stri
   const int t0 = q_start[s] + chunk * LTC_CHUNK;
   const int n = min(LTC_CHUNK, q_start[s + 1] - t0);
   if (n <= 0) return;
-  const float l2 = log2f(decay[h]);
-  ltc_stage_rows<D, D>(sm.q, q, stride, t0, n, h, 0, wide != 0);
-  ltc_stage_rows<D, D>(sm.k, k, stride, t0, n, h, 0, wide != 0);
-  ltc_stage_rows<DVB, DV>(sm.v, v, stride, t0, n, h, cb, wide != 0);
-  const float* s0 = work + ((size_t)blockIdx.y * heads + h) * D * DV;      // the chunk's start state [i][c]
+  const float l2 = STEPS ? 0.f : log2f(decay[h]);
+  const int hk = STEPS ? h / steps.per : h;
+  if (STEPS) ltc_factors(fac, steps, t0, n, h, heads);
+  ltc_stage_rows<D, STEPS>(sm.q, q, stride, t0, n, hk, d, 0, wide != 0);
+  ltc_stage_rows<D, STEPS>(sm.k, k, stride, t0, n, hk, d, 0, wide != 0);
+  ltc_stage_rows<DVB, STEPS>(sm.v, v, stride, t0, n, h, dv, cb, wide != 0);
+  const float* s0 = work + ((size_t)blockIdx.y * heads + h) * d * dv;      // the chunk's start state [i][c]
+  const bool whole = d == D && dv == DV;
 #pragma unroll 8
   for (int e0 = 0; e0 < D * DVB; e0 += LTC_THREADS * 4) {
     const int e = e0 + threadIdx.x * 4;
     const int i = e / DVB, c = e - i * DVB;
-    const float4 x = *(const float4*)(s0 + (size_t)i * DV + cb + c);
-    float hi[4] = {x.x, x.y, x.z, x.w}, lo[4];
+    float hi[4], lo[4];
+    if (whole) {
+      const float4 x = *(const float4*)(s0 + (size_t)i * DV + cb + c);
+      hi[0] = x.x; hi[1] = x.y; hi[2] = x.z; hi[3] = x.w;
+    } else {
+#pragma unroll
+      for (int y = 0; y < 4; ++y) hi[y] = (i < d && cb + c + y < dv) ? s0[(size_t)i * dv + cb + c + y] : 0.f;
+    }
 #pragma unroll
     for (int y = 0; y < 4; ++y) {
       const float r = __bfloat162float(__float2bfloat16_rn(hi[y]));
@@ -237,7 +294,8 @@ lightning_mma_pass2_kernel(const bf16* q, const bf16* k, const bf16* v, int stri
       tgm_mma(o[2 * np + 1], a, bl[2], bl[3]);
     }
   }
-  const float up = ltc_pow(l2, r0 + g + 1), dn = ltc_pow(l2, r0 + g + 9);
+  const float up = STEPS ? exp2f(fac.L[r0 + g]) : ltc_pow(l2, r0 + g + 1);
+  const float dn = STEPS ? exp2f(fac.L[r0 + g + 8]) : ltc_pow(l2, r0 + g + 9);
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt) {
     o[nt][0] *= up; o[nt][1] *= up;
@@ -268,7 +326,8 @@ lightning_mma_pass2_kernel(const bf16* q, const bf16* k, const bf16* v, int stri
 #pragma unroll
     for (int x = 0; x < 4; ++x) {
       const int t = r0 + g + 8 * (x >> 1), j = nt * 8 + 2 * tq + (x & 1);
-      p[nt][x] = (j <= t) ? p[nt][x] * ltc_pow(l2, t - j) : 0.f;
+      if (STEPS) p[nt][x] = (j <= t) ? p[nt][x] * (exp2f(fac.L[t] - fac.L[j]) * fac.dt[j]) : 0.f;
+      else p[nt][x] = (j <= t) ? p[nt][x] * ltc_pow(l2, t - j) : 0.f;
     }
   // weights times values, the weights as value + remainder
 #pragma unroll
@@ -298,31 +357,37 @@ lightning_mma_pass2_kernel(const bf16* q, const bf16* k, const bf16* v, int stri
   for (int nt = 0; nt < NT; ++nt) {
     const int c = cb + cbase + nt * 8 + 2 * tq;
     const int ta = r0 + g, tb = r0 + g + 8;
-    if (ta < n) *(float2*)(out + ((size_t)(t0 + ta) * heads + h) * DV + c) = make_float2(o[nt][0], o[nt][1]);
-    if (tb < n) *(float2*)(out + ((size_t)(t0 + tb) * heads + h) * DV + c) = make_float2(o[nt][2], o[nt][3]);
+    if (STEPS) {
+      const float skip = steps.skip[h];
+      const int cv = cbase + nt * 8 + 2 * tq;
+      o[nt][0] = fmaf(skip, to_f32(sm.v[ta][cv]), o[nt][0]); o[nt][1] = fmaf(skip, to_f32(sm.v[ta][cv + 1]), o[nt][1]);
+      o[nt][2] = fmaf(skip, to_f32(sm.v[tb][cv]), o[nt][2]); o[nt][3] = fmaf(skip, to_f32(sm.v[tb][cv + 1]), o[nt][3]);
+    }
+    if (ta < n) ltc_put2(out + ((size_t)(t0 + ta) * heads + h) * dv, 0, c, 1, dv, o[nt][0], o[nt][1]);
+    if (tb < n) ltc_put2(out + ((size_t)(t0 + tb) * heads + h) * dv, 0, c, 1, dv, o[nt][2], o[nt][3]);
   }
 }
 
 // Launches the two passes around `chain` (the caller's kernel that turns end-from-zero states into start
 // states).  Returns false if this head shape is not instantiated.
-template <int D, int DV, typename Chain>
-static bool ltc_launch(const bf16* q, const bf16* k, const bf16* v, int stride, const float* decay, float* work,
-                       const int* q_start, int num_seqs, int max_chunks, float* out, int heads, cudaStream_t stream,
-                       Chain chain) {
+template <int D, int DV, bool STEPS, typename Chain>
+static bool ltc_launch(const bf16* q, const bf16* k, const bf16* v, int stride, const float* decay, LtSteps steps,
+                       float* work, const int* q_start, int num_seqs, int max_chunks, float* out, int heads, int d,
+                       int dv, cudaStream_t stream, Chain chain) {
   const dim3 grid(heads, num_seqs * max_chunks);
   const size_t s1 = sizeof(LtcSmem1<D, DV>), s2 = sizeof(LtcSmem2<D, DV / LtcSplit<D, DV>::N>);
   static bool allowed = false;
   if (!allowed) {
-    cudaFuncSetAttribute(lightning_mma_pass1_kernel<D, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
-    cudaFuncSetAttribute(lightning_mma_pass2_kernel<D, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
+    cudaFuncSetAttribute(lightning_mma_pass1_kernel<D, DV, STEPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
+    cudaFuncSetAttribute(lightning_mma_pass2_kernel<D, DV, STEPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
     allowed = true;
   }
   // rows that start on 8-byte boundaries are fetched four values a load
-  const int wide = stride % 4 == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 7) == 0;
-  rllm_launch_pdl(lightning_mma_pass1_kernel<D, DV>, grid, dim3(LTC_THREADS), s1, stream, k, v, stride, wide, decay, work,
-                  q_start, max_chunks, heads);
+  const int wide = stride % 4 == 0 && d % 4 == 0 && dv % 4 == 0 && (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v) & 7) == 0;
+  rllm_launch_pdl(lightning_mma_pass1_kernel<D, DV, STEPS>, grid, dim3(LTC_THREADS), s1, stream, k, v, stride, wide, decay,
+                  steps, work, q_start, max_chunks, heads, d, dv);
   chain();
-  rllm_launch_pdl(lightning_mma_pass2_kernel<D, DV>, dim3(grid.x, grid.y, LtcSplit<D, DV>::N), dim3(LTC_THREADS), s2, stream, q, k, v, stride, wide, decay,
-                  (const float*)work, q_start, max_chunks, out, heads);
+  rllm_launch_pdl(lightning_mma_pass2_kernel<D, DV, STEPS>, dim3(grid.x, grid.y, LtcSplit<D, DV>::N), dim3(LTC_THREADS), s2, stream, q, k, v, stride, wide, decay,
+                  steps, (const float*)work, q_start, max_chunks, out, heads, d, dv);
   return true;
 }

@@ -15,7 +15,8 @@
 //                        weights (queries and keys are divided by their root mean square and nothing
 //                        else).  `qt_every` > 0: a query at position p is multiplied by
 //                        1 + qt_coef * ln(floor((p + 1) / qt_every) + 1), a temperature that grows with
-//                        the position; keys are not.
+//                        the position; keys are not.  `row_norm`: one root mean square over all of a token's
+//                        queries and one over all its keys, weights [nq dk] and [nkv dk] (a block a token).
 //   rms_mean             out = (1/n) sum_i rms(x_i) * w_i  over n = 2 inputs of one width
 //                        (branches of a mixer that run side by side)
 //   gated_rmsnorm        out = rms(x) * w * sigmoid(g)     (x float32, g in the activation dtype)
@@ -26,6 +27,38 @@
 #include <math.h>
 
 #define HN_WARPS 4
+
+// One query or key head after its norm: dst (or src itself where dst is null) gets (src + bs) * r * w, its first rd
+// dims rotated; r and w only where `scaled`.  A lane reads both members of its pairs before it writes them, and no
+// other lane touches them: in place is safe.
+template <typename T, typename TW>
+__device__ __forceinline__ void hn_scale_rotate(T* src, T* dst, const float* bs, const TW* w, bool scaled, float r,
+                                                int pos, const double* __restrict__ inv_freq, int rd, float mag, int dk,
+                                                int dkp, int lane) {
+  T* o = dst ? dst : src;
+  const int half = rd >> 1;
+  for (int i = lane; i < half; i += 32) {
+    float a = to_f32(src[i]) + (bs ? bs[i] : 0.f), b = to_f32(src[i + half]) + (bs ? bs[i + half] : 0.f);
+    if (scaled) { a *= r * (w ? to_f32(w[i]) : 1.0f); b *= r * (w ? to_f32(w[i + half]) : 1.0f); }
+    float c, sn;
+    if (sizeof(T) == 4) {
+      double sd, cd;
+      sincos((double)pos * inv_freq[i], &sd, &cd);
+      c = (float)(cd * (double)mag); sn = (float)(sd * (double)mag);
+    } else {
+      rope_cos_sin(pos, inv_freq[i], &c, &sn);
+      c *= mag; sn *= mag;
+    }
+    o[i] = from_f32<T>(a * c - b * sn);
+    o[i + half] = from_f32<T>(b * c + a * sn);
+  }
+  for (int i = rd + lane; i < (dst ? dkp : dk); i += 32) {
+    if (i >= dk) { o[i] = from_f32<T>(0.f); continue; }
+    float a = to_f32(src[i]) + (bs ? bs[i] : 0.f);
+    if (scaled) a *= r * (w ? to_f32(w[i]) : 1.0f);
+    o[i] = from_f32<T>(a);
+  }
+}
 
 // qkv: T rows of [nq * dk | nkv * dk | nkv * dv] with row stride `stride`.
 template <typename T, typename TW>
@@ -84,29 +117,50 @@ head_norm_kv_write_kernel(T* qkv, int stride, const int* positions, const int* t
     r = 1.0f / sqrtf(ss / (float)dk + eps);
   }
   if (warm) r *= 1.0f + qt_coef * logf((float)((pos + 1) / qt_every) + 1.0f);
-  T* o = dst ? dst : src;
-  const int half = rd >> 1;
-  // a lane reads both members of its pairs before it writes them, and no other lane touches them: in place is safe
-  for (int i = lane; i < half; i += 32) {
-    float a = to_f32(src[i]) + (bs ? bs[i] : 0.f), b = to_f32(src[i + half]) + (bs ? bs[i + half] : 0.f);
-    if (scaled) { a *= r * (w ? to_f32(w[i]) : 1.0f); b *= r * (w ? to_f32(w[i + half]) : 1.0f); }
-    float c, sn;
-    if (sizeof(T) == 4) {
-      double sd, cd;
-      sincos((double)pos * inv_freq[i], &sd, &cd);
-      c = (float)(cd * (double)mag); sn = (float)(sd * (double)mag);
-    } else {
-      rope_cos_sin(pos, inv_freq[i], &c, &sn);
-      c *= mag; sn *= mag;
+  hn_scale_rotate(src, dst, bs, w, scaled, r, pos, inv_freq, rd, mag, dk, dkp, lane);
+}
+
+// The same where the norm runs over a token's whole row of queries, and over its whole row of keys: weights
+// [nq * dk] and [nkv * dk].  One block a token.
+template <typename T, typename TW>
+__global__ void __launch_bounds__(256)
+row_norm_kv_write_kernel(T* qkv, int stride, const int* positions, const int* token_seq, const TW* wq, const TW* wk,
+                         float eps, const int* block_table, int max_blocks, T* kcache, T* vcache, int nq, int nkv,
+                         int dk, int dv, int dkp, int dvp, T* q_out, int page_size, int num_pages, int write_kv,
+                         const float* __restrict__ bias, const double* __restrict__ inv_freq, int rd, float mag,
+                         float qt_coef, int qt_every, int* err) {
+  __shared__ float red[32];
+  pdl_wait();
+  pdl_launch();
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  T* row = qkv + (size_t)t * stride;
+  const int pos = positions[t];
+  const int blk = pos / page_size;
+  const int page = blk < max_blocks ? block_table[(size_t)token_seq[t] * max_blocks + blk] : -1;
+  const bool place = write_kv && page >= 0 && page < num_pages;
+  if (write_kv && !place && threadIdx.x == 0) atomicOr(err, 2);
+  float sq = 0.f, sk = 0.f;
+  for (int i = threadIdx.x; i < nq * dk; i += blockDim.x) { const float v = to_f32(row[i]) + (bias ? bias[i] : 0.f); sq = fmaf(v, v, sq); }
+  for (int i = nq * dk + threadIdx.x; i < (nq + nkv) * dk; i += blockDim.x) { const float v = to_f32(row[i]) + (bias ? bias[i] : 0.f); sk = fmaf(v, v, sk); }
+  sq = block_sum(sq, red);
+  sk = block_sum(sk, red);                              // (behind its barriers every query element has been read)
+  float rq = 1.0f / sqrtf(sq / (float)(nq * dk) + eps);
+  const float rk = 1.0f / sqrtf(sk / (float)(nkv * dk) + eps);
+  if (qt_every > 0) rq *= 1.0f + qt_coef * logf((float)((pos + 1) / qt_every) + 1.0f);
+  for (int h = warp; h < nq + (place ? 2 * nkv : 0); h += warps) {
+    if (h >= nq + nkv) {                                // a value head: copied (with its bias)
+      const size_t at = (size_t)(nq + nkv) * dk + (size_t)(h - nq - nkv) * dv;
+      T* dst = vcache + (((size_t)page * nkv + h - nq - nkv) * page_size + pos % page_size) * dvp;
+      for (int i = lane; i < dvp; i += 32)
+        dst[i] = (i >= dv) ? from_f32<T>(0.f) : (bias ? from_f32<T>(to_f32(row[at + i]) + bias[at + i]) : row[at + i]);
+      continue;
     }
-    o[i] = from_f32<T>(a * c - b * sn);
-    o[i + half] = from_f32<T>(b * c + a * sn);
-  }
-  for (int i = rd + lane; i < (dst ? dkp : dk); i += 32) {
-    if (i >= dk) { o[i] = from_f32<T>(0.f); continue; }
-    float a = to_f32(src[i]) + (bs ? bs[i] : 0.f);
-    if (scaled) a *= r * (w ? to_f32(w[i]) : 1.0f);
-    o[i] = from_f32<T>(a);
+    const bool is_q = h < nq;
+    T* dst = is_q ? (q_out ? q_out + ((size_t)t * nq + h) * dkp : nullptr)
+                  : kcache + (((size_t)page * nkv + h - nq) * page_size + pos % page_size) * dkp;
+    const TW* w = is_q ? wq + (size_t)h * dk : wk + (size_t)(h - nq) * dk;
+    hn_scale_rotate(row + (size_t)h * dk, dst, bias ? bias + (size_t)h * dk : nullptr, w, true, is_q ? rq : rk, pos,
+                    inv_freq, rd, mag, dk, dkp, lane);
   }
 }
 
@@ -194,7 +248,8 @@ RLLM_EXPORT int rllm_head_norm_kv_write(void* qkv, int dtype, int stride, const 
                                         int max_blocks, void* kcache, void* vcache, int T, int nq, int nkv, int dk,
                                         int dv, int dkp, int dvp, void* q_out, int page_size, int num_pages,
                                         int write_kv, const float* bias, const double* inv_freq, int rd, float mag,
-                                        int unit_norm, float qt_coef, int qt_every, int* err, cudaStream_t stream) {
+                                        int unit_norm, float qt_coef, int qt_every, int row_norm, int* err,
+                                        cudaStream_t stream) {
   if (T <= 0) return 0;
   if (nq <= 0 || nkv < 0 || dk <= 0 || dv <= 0 || dkp < dk || dvp < dv) return RLLM_E_BADARG;
   if (rd < 0 || rd > dk || (rd & 1) || (rd > 0 && !inv_freq)) return RLLM_E_BADARG;
@@ -210,6 +265,16 @@ RLLM_EXPORT int rllm_head_norm_kv_write(void* qkv, int dtype, int stride, const 
                                      stride, positions, token_seq, block_table, max_blocks, (bf16*)kcache, (bf16*)vcache,
                                      T, nq, nkv_w, dk, dv, page_size, num_pages, write_kv, bias, inv_freq, rd, mag, err);
     return (int)e8;
+  }
+  if (row_norm) {
+    if (!wq || !wk || nkv <= 0 || page_size <= 0) return RLLM_E_BADARG;
+    RLLM_DISPATCH_DTYPE(dtype, TT, RLLM_DISPATCH_DTYPE(w_dtype, TW,
+      (rllm_launch_pdl(row_norm_kv_write_kernel<TT, TW>, dim3(T), dim3(256), (size_t)0, stream, (TT*)qkv, stride, positions,
+                       token_seq, (const TW*)wq, (const TW*)wk, eps, block_table, max_blocks, (TT*)kcache, (TT*)vcache,
+                       nq, nkv, dk, dv, dkp, dvp, (TT*)q_out, page_size, num_pages, write_kv, bias, inv_freq, rd, mag,
+                       qt_coef, qt_every, err))));
+    RLLM_LAUNCH_CHECK();
+    return 0;
   }
   const long long warps = (long long)T * (nq + 2 * nkv);
   const unsigned blocks = (unsigned)((warps + HN_WARPS - 1) / HN_WARPS);

@@ -1,6 +1,6 @@
 // The selective state-space recurrence (Mamba) and the short causal convolution ahead of it.
 //
-//   convolution: c_t = silu(bias + sum_j w[ch, j] x_{t - (taps - 1) + j})   per channel, zeros before the
+//   convolution: c_t = silu(bias + sum_j w[ch, j] x_{t - (taps - 1) + j})   per channel (the bias may be absent), zeros before the
 //                sequence's start; the last taps - 1 inputs are per-request state (float32 [taps - 1, E])
 //   recurrence:  dt = softplus(r_t + dt_bias)     (r_t: the token's step projection, one per channel)
 //                S[ch, n] <- exp(dt A[ch, n]) S[ch, n] + dt c_t B_t[n],   A = -exp(A_log)
@@ -44,7 +44,7 @@ causal_conv_kernel(const T* x, int stride, const TW* w, const TW* bias, float* t
   }
   float* tl = tail + (size_t)slot * (taps - 1) * E + c;
   const int li = t - first;
-  float acc = to_f32(bias[c]);
+  float acc = bias ? to_f32(bias[c]) : 0.f;
   for (int j = 0; j < taps; ++j) {
     const int src = li - (taps - 1) + j;
     const float v = (src >= 0) ? to_f32(x[(size_t)(first + src) * stride + c]) : tl[(size_t)(taps - 1 + src) * E];
@@ -73,7 +73,7 @@ causal_conv_run_kernel(const T* x, int stride, const TW* w, const TW* bias, floa
   float wv[CV_TAPS];
 #pragma unroll
   for (int k = 0; k < CV_TAPS; ++k) wv[CV_TAPS - 1 - k] = (mine && k < taps) ? to_f32(w[(size_t)c * taps + taps - 1 - k]) : 0.f;
-  const float b = mine ? to_f32(bias[c]) : 0.f;
+  const float b = (mine && bias) ? to_f32(bias[c]) : 0.f;
   pdl_wait();
   pdl_launch();
   if (!mine) return;

@@ -730,6 +730,50 @@ def gated_postnorm_add(x_in: torch.Tensor, x_out: torch.Tensor, y: torch.Tensor,
     return nxt
 
 
+def postnorm_add(x: torch.Tensor, y, weight: torch.Tensor, eps: float, multiplier: float,
+                 act_dtype: torch.dtype) -> torch.Tensor:
+    """x += multiplier * rmsnorm(y) * weight in place (x float32 [T, H]; y [T, H] in the activation dtype, or a
+    ``WeightedSum`` of two such terms, added up in float32 before the norm).  Returns the new x in the activation
+    dtype (x itself for float32)."""
+    lib = build.load_library("layer_glue")
+    terms, scales = ((y,), (1.0, 0.0)) if isinstance(y, torch.Tensor) else (tuple(y.terms), tuple(y.scales))
+    T, H = x.shape
+    assert x.dtype is torch.float32 and weight.numel() == H
+    _contig(x, "x"); _contig(weight, "weight")
+    for t in terms:
+        assert t.shape == (T, H) and t.dtype is act_dtype
+        _contig(t, "y")
+    out = None if act_dtype is torch.float32 else torch.empty((T, H), dtype=act_dtype, device=x.device)
+    _check(lib.rllm_postnorm_add(_ptr(x), _ptr(terms[0]), _ptr(terms[1] if len(terms) > 1 else None),
+                                 c_float(scales[0]), c_float(scales[1]), _ptr(weight), c_float(eps),
+                                 c_float(multiplier), _ptr(out), c_int(T), c_int(H), c_int(dtype_code(act_dtype)),
+                                 c_int(dtype_code(weight.dtype)), _stream()), "postnorm_add")
+    return x if out is None else out
+
+
+def activation_rows(x: torch.Tensor, act_dtype: torch.dtype) -> torch.Tensor:
+    """The float32 stream in the activation dtype (itself for float32)."""
+    assert x.dtype is torch.float32
+    if act_dtype is torch.float32:
+        return x
+    lib = build.load_library("layer_glue")
+    _contig(x, "x")
+    out = torch.empty(x.shape, dtype=act_dtype, device=x.device)
+    _check(lib.rllm_activation_rows(_ptr(x), _ptr(out), c_longlong(x.numel()), _stream()), "activation_rows")
+    return out
+
+
+def scaled_sum2(a: torch.Tensor, b: torch.Tensor, scale_a: float, scale_b: float) -> torch.Tensor:
+    """scale_a * a + scale_b * b, added in float32."""
+    lib = build.load_library("layer_glue")
+    assert a.shape == b.shape and a.dtype is b.dtype
+    _contig(a, "a"); _contig(b, "b")
+    out = torch.empty_like(a)
+    _check(lib.rllm_scaled_sum2(_ptr(a), _ptr(b), c_float(scale_a), c_float(scale_b), _ptr(out),
+                                c_int(dtype_code(a.dtype)), c_longlong(a.numel()), _stream()), "scaled_sum2")
+    return out
+
+
 def depth_average(history: torch.Tensor, levels: int, coeff: torch.Tensor, stream_out: Optional[torch.Tensor],
                   norm_weight: Optional[torch.Tensor], eps: float, act_dtype: torch.dtype,
                   rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
@@ -1157,7 +1201,7 @@ def head_norm_kv_write(qkv: torch.Tensor, positions: torch.Tensor, token_seq: to
                        dk: int, dv: int, err: torch.Tensor, write_kv: bool = True,
                        q_out: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
                        inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, magnitude: float = 1.0,
-                       unit_norm: bool = False, q_temp=None) -> None:
+                       unit_norm: bool = False, q_temp=None, row_norm: bool = False) -> None:
     """qkv [T, nq dk + nkv dk + nkv dv]: every query head (in place) and key head is divided by its root mean
     square and multiplied by the weight [dk] (None: left as it is); keys and values go to the token's place in
     kcache [pages, nkv, page, dkp] and vcache [pages, nkv, page, dvp].  Cache rows wider than the heads (dkp > dk,
@@ -1166,8 +1210,9 @@ def head_norm_kv_write(qkv: torch.Tensor, positions: torch.Tensor, token_seq: to
     with ``rotary_dim`` > 0 rotates the first rotary_dim dims of every query and key head by the token's position
     (dimension i with i + rotary_dim / 2), cosine and sine times ``magnitude``.  ``unit_norm``: the heads are
     divided by their root mean square although there are no weights.  ``q_temp`` = (coef, every): a query at
-    position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).  Columns of qkv behind the
-    value heads are left alone."""
+    position p is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1).  ``row_norm``: one root mean square over all
+    of a token's queries and one over its keys, with weights [nq dk] and [nkv dk] (it wants ``write_kv``).  Columns of
+    qkv behind the value heads are left alone."""
     lib = build.load_library("mixer_glue")
     T = qkv.shape[0]
     assert qkv.shape[1] >= nq * dk + nkv * (dk + dv) and qkv.stride(1) == 1
@@ -1181,7 +1226,9 @@ def head_norm_kv_write(qkv: torch.Tensor, positions: torch.Tensor, token_seq: to
         assert q_out.shape == (T, nq * dkp) and q_out.dtype is qkv.dtype and q_out.is_contiguous()
     wd = q_weight.dtype if q_weight is not None else torch.float32
     if q_weight is not None:
-        assert k_weight is not None and k_weight.dtype is wd and q_weight.numel() == dk and k_weight.numel() == dk
+        nw, kw = (nq * dk, nkv * dk) if row_norm else (dk, dk)
+        assert k_weight is not None and k_weight.dtype is wd and q_weight.numel() == nw and k_weight.numel() == kw
+    assert not row_norm or (q_weight is not None and write_kv)
     if write_kv:
         dvp = vcache.shape[3]
         assert kcache.dtype is qkv.dtype and vcache.dtype is qkv.dtype and kcache.shape[3] == dkp and dvp >= dv
@@ -1198,7 +1245,7 @@ def head_norm_kv_write(qkv: torch.Tensor, positions: torch.Tensor, token_seq: to
                                        c_int(page_size), c_int(pages), c_int(1 if write_kv else 0), _ptr(bias),
                                        _ptr(inv_freq if rotary_dim else None), c_int(rotary_dim), c_float(magnitude),
                                        c_int(1 if unit_norm else 0), c_float(q_temp[0] if q_temp else 0.0),
-                                       c_int(int(q_temp[1]) if q_temp else 0),
+                                       c_int(int(q_temp[1]) if q_temp else 0), c_int(1 if row_norm else 0),
                                        _ptr(err), _stream()), "head_norm_kv_write")
 
 
@@ -1295,18 +1342,19 @@ def lightning_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: tor
     return out
 
 
-def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, tail: torch.Tensor,
+def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], tail: torch.Tensor,
                 q_start: torch.Tensor, token_seq: torch.Tensor, slots: torch.Tensor, num_seqs: int,
                 any_long: bool, err: torch.Tensor) -> torch.Tensor:
-    """silu(bias + causal convolution per channel); x [T, E] (a column slice will do); weight [E, taps], the
+    """silu(bias + causal convolution per channel; ``bias`` may be None); x [T, E] (a column slice will do); weight [E, taps], the
     last column the current token's; tail float32 [slots, taps - 1, E]: a request's last inputs, read for the
     places before this step and moved on.  ``any_long``: some sequence brings more than one token."""
     lib = build.load_library("selective_scan")
     T, E = x.shape
     taps = weight.shape[1]
-    assert weight.shape == (E, taps) and bias.numel() == E and weight.dtype is bias.dtype and x.stride(1) == 1
+    assert weight.shape == (E, taps) and x.stride(1) == 1
+    assert bias is None or (bias.numel() == E and weight.dtype is bias.dtype and bias.is_contiguous())
     assert tail.dtype is torch.float32 and tuple(tail.shape[1:]) == (max(taps - 1, 0), E)
-    _contig(weight, "weight"); _contig(bias, "bias"); _contig(tail, "tail")
+    _contig(weight, "weight"); _contig(tail, "tail")
     out = torch.empty((T, E), dtype=x.dtype, device=x.device)
     _check(lib.rllm_causal_conv(_ptr(x), c_int(x.stride(0)), c_int(dtype_code(x.dtype)), _ptr(weight), _ptr(bias),
                                 c_int(dtype_code(weight.dtype)), _ptr(tail), _ptr(q_start), _ptr(token_seq),
@@ -1459,4 +1507,89 @@ def head_gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor
                                        _ptr(weight), c_int(dtype_code(weight.dtype)), _ptr(out),
                                        c_int(dtype_code(out_dtype)), c_int(T), c_int(heads), c_int(W // heads),
                                        c_float(eps), _stream()), "head_gated_rmsnorm")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# the state-space recurrence (ssd.cu)
+# ---------------------------------------------------------------------------
+def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor,
+             state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, num_seqs: int, heads: int, groups: int,
+             n: int, p: int, err: torch.Tensor, max_q_len: int = 1) -> torch.Tensor:
+    """The Mamba-2 recurrence over this step's tokens.  xbc [T, heads p + 2 groups n]: x | B | C, activated; dt
+    float32 [T, heads]: the steps before bias and softplus; dt_bias, a_log, skip float32 [heads]; state float32
+    [slots, heads, n, p], updated in place.  Returns y = S^T C + skip x, float32 [T, heads p].  Portions long enough
+    to fill the GPU with chunks are scanned as chunks side by side; the result differs by rounding only."""
+    lib = build.load_library("ssd")
+    T = xbc.shape[0]
+    assert xbc.shape[1] == heads * p + 2 * groups * n and xbc.stride(1) == 1
+    assert dt.dtype is torch.float32 and dt.shape == (T, heads)
+    for t, name in ((dt_bias, "dt_bias"), (a_log, "a_log"), (skip, "skip")):
+        assert t.dtype is torch.float32 and t.numel() == heads
+        _contig(t, name)
+    assert state.dtype is torch.float32 and tuple(state.shape[1:]) == (heads, n, p)
+    _contig(dt, "dt"); _contig(state, "state")
+    out = torch.empty((T, heads * p), dtype=torch.float32, device=xbc.device)
+    chunks = _chunks_for(int(lib.rllm_ssd_chunk()), max_q_len, num_seqs)
+    work = torch.empty(num_seqs * chunks * heads * (n * p + 1), dtype=torch.float32, device=xbc.device) if chunks else None
+    chunk_dt = work[num_seqs * chunks * heads * n * p:] if chunks else None
+    _check(lib.rllm_ssd_scan(_ptr(xbc), c_int(xbc.stride(0) if T > 1 else xbc.shape[1]), c_int(dtype_code(xbc.dtype)),
+                             _ptr(dt), _ptr(dt_bias), _ptr(a_log), _ptr(skip), _ptr(state), _ptr(work), _ptr(chunk_dt),
+                             _ptr(q_start), _ptr(slots), c_int(state.shape[0]), c_int(num_seqs), c_int(chunks),
+                             _ptr(out), c_int(heads), c_int(groups), c_int(n), c_int(p), _ptr(err), _stream()),
+           "ssd_scan")
+    return out
+
+
+def silu_gated_group_rmsnorm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, groups: int,
+                             out_dtype: torch.dtype) -> torch.Tensor:
+    """v = y * silu(z); each of ``groups`` equal parts of a row over its own root mean square, times weight.
+    y float32 [T, E]; z [T, E] in ``out_dtype`` (may be a column slice); weight float32 [E]."""
+    lib = build.load_library("ssd")
+    T, E = y.shape
+    assert y.dtype is torch.float32 and weight.dtype is torch.float32 and weight.numel() == E
+    assert z.shape == (T, E) and z.dtype is out_dtype and z.stride(1) == 1
+    _contig(y, "y"); _contig(weight, "weight")
+    out = torch.empty((T, E), dtype=out_dtype, device=y.device)
+    _check(lib.rllm_silu_gated_group_rmsnorm(_ptr(y), _ptr(z), c_int(z.stride(0) if T > 1 else max(E, z.stride(0))),
+                                             _ptr(weight), _ptr(out), c_int(dtype_code(out_dtype)), c_int(T), c_int(E),
+                                             c_int(groups), c_float(eps), _stream()), "silu_gated_group_rmsnorm")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# the gated delta rule with a decay per key channel (channel_delta.cu)
+# ---------------------------------------------------------------------------
+def channel_delta_scan(c: torch.Tensor, step: torch.Tensor, b: torch.Tensor, dt_bias: torch.Tensor,
+                       a_log: torch.Tensor, unit_eps: float, state: torch.Tensor, q_start: torch.Tensor,
+                       slots: torch.Tensor, num_seqs: int, heads: int, kv: int, d: int, dv: int,
+                       err: torch.Tensor) -> torch.Tensor:
+    """The delta rule over this step's tokens of every sequence, in order, from and into the sequences' slots.
+    c [T, 2 kv d + heads dv]: q | k | v after their convolutions; step float32 [T, heads d]: the decays' step
+    before bias and softplus; b float32 [T, heads]: beta before its sigmoid; dt_bias float32 [heads d], a_log
+    float32 [heads]; state float32 [slots, heads, d, dv].  q and k are made unit vectors (``unit_eps`` under the
+    root), q is multiplied by d^(-1/2).  Returns o float32 [T, heads dv]."""
+    lib = build.load_library("channel_delta")
+    T = c.shape[0]
+    assert c.shape[1] == 2 * kv * d + heads * dv and c.stride(1) == 1
+    assert step.dtype is torch.float32 and step.shape == (T, heads * d)
+    assert b.dtype is torch.float32 and b.shape == (T, heads)
+    assert dt_bias.dtype is torch.float32 and dt_bias.numel() == heads * d
+    assert a_log.dtype is torch.float32 and a_log.numel() == heads
+    assert state.dtype is torch.float32 and tuple(state.shape[1:]) == (heads, d, dv)
+    for t, name in ((step, "step"), (b, "b"), (dt_bias, "dt_bias"), (a_log, "a_log"), (state, "state")):
+        _contig(t, name)
+    f32 = dict(dtype=torch.float32, device=c.device)
+    qn, kn, g = torch.empty((T, kv, d), **f32), torch.empty((T, kv, d), **f32), torch.empty((T, heads, d), **f32)
+    beta, out = torch.empty((T, heads), **f32), torch.empty((T, heads * dv), **f32)
+    stride = c.stride(0) if T > 1 else c.shape[1]
+    _check(lib.rllm_channel_delta_prepare(_ptr(c), c_int(stride), c_int(dtype_code(c.dtype)), _ptr(step), _ptr(b),
+                                          _ptr(dt_bias), _ptr(a_log), _ptr(qn), _ptr(kn), _ptr(g), _ptr(beta), c_int(T),
+                                          c_int(heads), c_int(kv), c_int(d), c_float(unit_eps),
+                                          c_float(float(d) ** -0.5), _stream()), "channel_delta_prepare")
+    v = c[:, 2 * kv * d:]
+    _check(lib.rllm_channel_delta_walk(_ptr(qn), _ptr(kn), _ptr(g), _ptr(beta), _ptr(v), c_int(stride),
+                                       c_int(dtype_code(c.dtype)), _ptr(state), _ptr(q_start), _ptr(slots),
+                                       c_int(state.shape[0]), c_int(num_seqs), _ptr(out), c_int(heads), c_int(kv),
+                                       c_int(d), c_int(dv), _ptr(err), _stream()), "channel_delta_walk")
     return out

@@ -1,7 +1,7 @@
 """Parts a layer is put together from.  Importing the package registers the
 built-in kinds."""
-from . import (attention, block, gated_block, hyper_block, latent_attention, lightning, mingru, mlp, mlstm, norm,  # noqa: F401  (registration)
-               parallel, rotary, routed_experts, selective_scan)
+from . import (attention, block, channel_delta, gated_block, hyper_block, latent_attention, lightning, mingru, mlp, mlstm, norm,  # noqa: F401  (registration)
+               parallel, rotary, routed_experts, selective_scan, state_space)
 from .base import (FeedForward, KVCacheView, Mixer, Norm, Part, PositionEncoding, StateCacheView,
                    StepContext)
 from .registry import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITION_ENCODINGS, build_part,

@@ -39,7 +39,12 @@ added to the denominator); ``qk_norm_weights`` False (with ``qk_norm``): the hea
 mean square and multiplied by nothing; ``q_temp`` = (coef, every): the query at position p is multiplied by
 1 + coef * ln(floor((p + 1) / every) + 1) after its norm; ``distance_slopes`` = x: slope_h * (p - j) is taken
 off the scaled score of key j, with slope_h = 2^(-x (h + 1) / num_heads) for head h (a bias linear in the
-distance, steeper for the first heads).
+distance, steeper for the first heads); ``qk_norm_span`` "row" (with ``qk_norm``): one root mean square over
+all of a token's query heads together, and one over its key heads, with weights [num_heads * head_dim] and
+[num_kv_heads * head_dim] ("head", the default: per head).
+
+A position part that rotates pairs (2i, 2i + 1) is served by the same kernels, which rotate halves: the rows of
+W_q, W_k, their biases and norm weights are put into the part's ``half_order`` when they are loaded.
 
 params: hidden_size, num_heads, num_kv_heads, head_dim, window (None: all
 keys), scale (None: 1/sqrt(head_dim)), position (PartSpec), shares_kv (True:
@@ -89,6 +94,11 @@ class PagedAttention(Mixer):
         self.sinks = bool(p.get("sinks", False))
         self.zero_sinks = p.get("sinks") == "zero"
         self.qk_weights = bool(p.get("qk_norm_weights", True))
+        self.qk_row = p.get("qk_norm_span", "head") == "row"
+        if p.get("qk_norm_span", "head") not in ("head", "row"):
+            raise ValueError(f"qk_norm_span {p['qk_norm_span']!r}; known: 'head', 'row'")
+        if self.qk_row and (self.qk_eps is None or not self.qk_weights or self.shares_kv):
+            raise ValueError("qk_norm_span 'row' goes with qk_norm, its weights and keys of the run's own")
         qt = p.get("q_temp")
         self.q_temp = (float(qt[0]), int(qt[1])) if qt else None
         if self.q_temp is not None and self.q_temp[1] < 1:
@@ -112,7 +122,7 @@ class PagedAttention(Mixer):
         import os
         self.dp = max(self.d, self.dv)
         if self.d == self.dv or self.dp not in (16, 32, 64, 128) or self.nq // max(1, self.nkv) > 16 or \
-                self.masked or os.environ.get("RLLM_ATTENTION_PAD") == "0":
+                self.gate == "element" or os.environ.get("RLLM_ATTENTION_PAD") == "0":
             self.dp = 0
         if self.nq % self.nkv:
             raise ValueError(f"num_heads {self.nq} must be a multiple of num_kv_heads {self.nkv}")
@@ -130,8 +140,9 @@ class PagedAttention(Mixer):
         pos = p.get("position")
         self.position = build_part("position_encoding", pos if pos is not None else PartSpec.of("none"),
                                    prefix=prefix)
-        if getattr(self.position, "interleaved", False):
-            raise ValueError("this mixer's kernels rotate halves; an interleaved rotation is not among them")
+        self.pairs = bool(getattr(self.position, "interleaved", False))
+        if self.pairs and self.position.head_dim != self.d:
+            raise ValueError(f"the rotation is of heads of {self.position.head_dim}, the mixer's heads have {self.d}")
         if not self.plain and self.position.fused_rotary() is None:
             raise ValueError("attention through the pages takes a rotation that its kernel can apply, or none")
         if self.shares_kv and self.bias:
@@ -143,6 +154,7 @@ class PagedAttention(Mixer):
         self.b_qkv = self.b_o = self.sink = self.slopes = None
         self.w_qkv: Optional[torch.Tensor] = None
         self.w_o: Optional[torch.Tensor] = None
+        self._first_given = False
 
     # -- weights ----------------------------------------------------------
     def _names(self):
@@ -160,10 +172,11 @@ class PagedAttention(Mixer):
                       TensorSpec(v, (self.nkv * self.dv, self.hidden))]
         specs.append(TensorSpec(o, (self.hidden, self.nq * self.dv)))
         if self.qk_eps is not None and self.qk_weights:
-            specs.append(TensorSpec(self.prefix + self.names["q_norm"], (self.d,), role="vector",
+            nq, nkv = (self.nq, self.nkv) if self.qk_row else (1, 1)
+            specs.append(TensorSpec(self.prefix + self.names["q_norm"], (nq * self.d,), role="vector",
                                     init=("one_plus_normal", 0.1)))
             if not self.shares_kv:
-                specs.append(TensorSpec(self.prefix + self.names["k_norm"], (self.d,), role="vector",
+                specs.append(TensorSpec(self.prefix + self.names["k_norm"], (nkv * self.d,), role="vector",
                                         init=("one_plus_normal", 0.1)))
         if self.bias:
             for key, n in (("q_bias", self.nq * self.d), ("k_bias", self.nkv * self.d), ("v_bias", self.nkv * self.dv),
@@ -175,8 +188,22 @@ class PagedAttention(Mixer):
             specs.append(TensorSpec(self.prefix + self.names["g"], (self.gate_width, self.hidden)))
         return specs
 
+    def _halves(self, t: torch.Tensor) -> torch.Tensor:
+        """Rows (or elements) of query or key heads in the order in which rotating halves rotates the pairs."""
+        if not self.pairs:
+            return t
+        idx = torch.tensor(self.position.half_order(), dtype=torch.long, device=t.device)
+        return t.view(-1, self.d, *t.shape[1:]).index_select(1, idx).reshape(t.shape).contiguous()
+
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
         q, k, v, o = self._names()
+        self._first_given = False
+        if self.pairs:
+            tensors = dict(tensors)
+            for key in ("q", "k", "q_norm", "k_norm", "q_bias", "k_bias"):
+                name = self.prefix + self.names[key] if key in self.names else None
+                if name in tensors:
+                    tensors[name] = self._halves(tensors[name])
         if self.shares_kv:
             # with a gate [Wq; Wg]: the gate's pre-activations lie behind the query heads
             stack = [tensors[q]] + ([tensors[self.prefix + self.names["g"]]] if self.gate else [])
@@ -219,7 +246,7 @@ class PagedAttention(Mixer):
 
     def cache_need(self):
         if self.dp:
-            return KVPagesNeed(self.nkv, self.dp, self.window)
+            return KVPagesNeed(self.nkv, self.dp, self.window, keep_first=self.keep_first, chunk=self.chunk or None)
         return KVPagesNeed(self.nkv, self.d, self.window, v_dim=None if self.dv == self.d else self.dv,
                            keep_first=self.keep_first, chunk=self.chunk or None)
 
@@ -250,16 +277,17 @@ class PagedAttention(Mixer):
                                    self.w_kn, self.qk_eps or 0.0, table, cache.k, cache.v, self.nq,
                                    0 if self.shares_kv else self.nkv, self.d, self.dv, ctx.err, write_kv=writes,
                                    q_out=q_pad, bias=self.b_qkv, inv_freq=inv_freq, rotary_dim=rd, magnitude=mag,
-                                   unit_norm=self.qk_eps is not None and not self.qk_weights, q_temp=self.q_temp)
+                                   unit_norm=self.qk_eps is not None and not self.qk_weights, q_temp=self.q_temp,
+                                   row_norm=self.qk_row)
         d, dv = (self.dp, self.dp) if self.dp else (self.d, self.dv)
-        if q_pad is not None:
-            qkv = q_pad
-        out = torch.empty((T, self.nq * dv), dtype=qkv.dtype, device=qkv.device)
-        window, stride = int(self.window or 0), qkv.shape[1]
         gate = None
         if self.gate:
             at = self.nq * self.d + (0 if self.shares_kv else self.nkv * (self.d + self.dv))
             gate = qkv[:, at: at + self.gate_width]
+        if q_pad is not None:
+            qkv = q_pad
+        out = torch.empty((T, self.nq * dv), dtype=qkv.dtype, device=qkv.device)
+        window, stride = int(self.window or 0), qkv.stride(0)
         opts = dict(keep_first=self.keep_first, chunk=self.chunk, softcap=self.softcap, sinks=self.sink, gate=gate,
                     gate_per_head=self.gate == "head") if self.masked else {}
         if self.slopes is not None:
@@ -291,8 +319,19 @@ class PagedAttention(Mixer):
         stream (it then calls ``forward`` with ``add_output_bias=False``); None: there is none."""
         return self.b_o
 
-    def forward(self, x, ctx: StepContext, cache: KVCacheView, residual=None, add_output_bias: bool = True):
-        out = self.attend(linear(x, self.w_qkv), ctx, cache)          # qkv [T, (nq + 2 nkv) d (+ the gate's)]
+    def give_first_weight(self) -> Optional[torch.Tensor]:
+        if self.plain or self._first_given:
+            return None
+        w, self.w_qkv, self._first_given = self.w_qkv, None, True
+        return w
+
+    def take_back_first_weight(self, weight: torch.Tensor) -> None:
+        self.w_qkv, self._first_given = weight, False
+
+    def forward(self, x, ctx: StepContext, cache: KVCacheView, residual=None, add_output_bias: bool = True,
+                first: Optional[torch.Tensor] = None):
+        # qkv [T, (nq + 2 nkv) d (+ the gate's)]
+        out = self.attend(linear(x, self.w_qkv) if first is None else first, ctx, cache)
         y = linear(out, self.w_o, residual=residual)
         if self.b_o is not None and add_output_bias:
             ops.add_row_bias(y, self.b_o)

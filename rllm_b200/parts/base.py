@@ -108,6 +108,14 @@ class NormedRows:
 
 
 @dataclass
+class ActivationRows:
+    """h is complete, and ``x`` [T, H] is h itself in the activation dtype, for a block whose sublayers read the
+    stream without a norm; any other reader ignores it."""
+
+    x: torch.Tensor
+
+
+@dataclass
 class PreparedInput:
     """The stream is complete, and ``x`` [T, H] is already the first sublayer's input of the block ``key``
     (that block's own read of the stream and its first norm, in the activation dtype), prepared by the
@@ -125,6 +133,16 @@ class PendingSum:
 
     terms: Tuple[torch.Tensor, ...]
     bias: Optional[torch.Tensor] = None
+
+
+@dataclass
+class WeightedSum:
+    """A sublayer's result that has not been added up yet: ``scales[0] * terms[0] + scales[1] * terms[1]``
+    (terms [T, H] in the activation dtype).  A mixer hands one out (``forward_terms``) to a block whose next
+    kernel reads both terms anyway."""
+
+    terms: Tuple[torch.Tensor, torch.Tensor]
+    scales: Tuple[float, float]
 
 
 @dataclass
@@ -224,6 +242,16 @@ class Mixer(Part):
         first step is a matrix product over stacked weights appends it there and returns True; its
         ``forward(..., side=True)`` then returns (result, that product's extra columns [T, rows], a view)."""
         return False
+
+    def give_first_weight(self) -> Optional[torch.Tensor]:
+        """A mixer whose first step is a matrix product of its input may give that product's weight [rows, H]
+        away, once, to someone who computes several such products as one; ``forward(..., first=...)`` then gets
+        the product's columns (a view with the wider product's row stride).  None: it keeps its weight."""
+        return None
+
+    def take_back_first_weight(self, weight: torch.Tensor) -> None:
+        """The weight that ``give_first_weight`` gave away comes back unused."""
+        raise NotImplementedError
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache) -> torch.Tensor:
         raise NotImplementedError

@@ -14,6 +14,14 @@ the product that ends the mixer (and the feed-forward) adds into h itself and
 leaves what the next norm needs, and the product that follows the norm applies
 it (see ``RowSumsq`` and ``ScaledRows`` in ``parts/base.py``).
 
+``post_norm`` normalises what the sublayers give, not what they read:
+    x <- x + c norm_0(mixer(x)),   x <- x + c norm_1(ffn(x))
+with a constant c (the feed-forward may be absent).  The norm of a sublayer's
+result, the add and the copy of the new stream in the activation dtype, which the
+next sublayer reads, are one kernel (``ActivationRows`` hands that copy to the next
+block); a mixer whose result is a weighted sum of two may leave the sum to that
+kernel too (``WeightedSum``).
+
 ``parallel_residual`` has one norm that both sublayers read:
     u   = norm_0(x)
     out = x + (mixer(u) + ffn(u))
@@ -27,8 +35,10 @@ from typing import List, Optional, Tuple
 
 import torch
 
-from .base import FeedForward, Mixer, Norm, PendingSum, RowSumsq, StepContext
+from ..kernels import ops
+from .base import ActivationRows, FeedForward, Mixer, Norm, Part, PendingSum, RowSumsq, StepContext
 from .registry import register_part
+from .spec import PartSpec
 
 
 @register_part("block", "pre_norm")
@@ -89,7 +99,6 @@ class ParallelResidualBlock:
     def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache, next_norm=None):
         norm = self.norms[0]
         if isinstance(pending, PendingSum) and not getattr(norm, "takes_pending_sum", False):
-            from ..kernels import ops
             ops.add_rows(h, pending.terms, pending.bias)
             pending = None
         if isinstance(pending, (torch.Tensor, PendingSum)):
@@ -104,9 +113,52 @@ class ParallelResidualBlock:
         terms = (a,) if self.ffn is None else (a, self.ffn.forward(u))
         trace = ctx.extras.get("residual_trace")         # a list: the stream after every layer (a copy)
         if trace is not None or not getattr(next_norm, "takes_pending_sum", False):
-            from ..kernels import ops
             ops.add_rows(h, terms, bias)
             if trace is not None:
                 trace.append(h.clone())
             return h, None
         return h, PendingSum(terms, bias)
+
+
+@register_part("block", "post_norm")
+class PostNormBlock(Part):
+    """params: hidden_size, multiplier (c above; 1 if absent)."""
+    graph_safe = True
+
+    def __init__(self, mixer: Mixer, ffn: Optional[FeedForward], norms: List[Norm], spec: PartSpec, prefix: str = ""):
+        super().__init__(spec, prefix)
+        if len(norms) != 2:
+            raise ValueError("a post_norm block has two norms: of the mixer's result and of the feed-forward's")
+        if any(not hasattr(n, "weight") or not hasattr(n, "eps") for n in norms):
+            raise ValueError("a post_norm block fuses its norms: they must be RMS norms with a weight and eps")
+        self.mixer, self.ffn, self.norms = mixer, ffn, norms
+        p = spec.get()
+        self.hidden = int(p["hidden_size"])
+        self.multiplier = float(p.get("multiplier", 1.0))
+
+    def parts(self):
+        return [self, self.mixer, self.norms[0]] + ([self.ffn, self.norms[1]] if self.ffn is not None else [])
+
+    def ignored_tensors(self) -> List[str]:
+        """A layer without a feed-forward does not use its second norm: a file that carries it is no error."""
+        return [] if self.ffn is not None else [self.norms[1].name]
+
+    def _add(self, h: torch.Tensor, y, norm, act_dtype: torch.dtype) -> torch.Tensor:
+        """h += c norm(y), in place; returns the new h in the activation dtype."""
+        return ops.postnorm_add(h, y, norm.weight, norm.eps, self.multiplier, act_dtype)
+
+    def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache):
+        if isinstance(pending, torch.Tensor):
+            ops.residual_add(h, pending)                  # a block of another kind ahead left its last add to us
+        elif isinstance(pending, PendingSum):
+            ops.add_rows(h, pending.terms, pending.bias)
+        x = pending.x if isinstance(pending, ActivationRows) else ops.activation_rows(h, ctx.act_dtype)
+        terms = self.mixer.forward_terms(x, ctx, cache) if hasattr(self.mixer, "forward_terms") else None
+        y = terms if terms is not None else self.mixer.forward(x, ctx, cache)
+        x = self._add(h, y, self.norms[0], ctx.act_dtype)
+        if self.ffn is not None:
+            x = self._add(h, self.ffn.forward(x), self.norms[1], ctx.act_dtype)
+        trace = ctx.extras.get("residual_trace")          # a list: the stream after every layer (a copy)
+        if trace is not None:
+            trace.append(h.clone())
+        return h, ActivationRows(x)

@@ -15,6 +15,8 @@ pair i gets the blend r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) of the
 slowed frequency: f_i / factor * r_i + f_i * (1 - r_i); and cosine and sine
 are both multiplied by 0.1 ln(factor) + 1 (``Rotary.magnitude``; 1 otherwise).
 
+A third rule, ``kind`` "linear" (factor): every frequency is divided by factor.
+
 No table over positions is stored: the kernel computes cos and sin of
 position * f_i in float64 per token, which is what the reference's table holds
 (rope.rs:24-28), for any position.
@@ -37,6 +39,8 @@ def rotary_frequencies(rotary_dim: int, theta: float, scaling: Optional[dict]) -
     if not scaling:
         return freqs
     factor = float(scaling["factor"])
+    if scaling.get("kind") == "linear":
+        return [f / factor for f in freqs]
     if scaling.get("kind") == "yarn":
         orig, theta = float(scaling["original"]), float(theta)
 
@@ -71,7 +75,8 @@ class Rotary(PositionEncoding):
     """params: head_dim, rotary_dim (<= head_dim, even), theta, scaling (dict or None),
     interleaved (False: dimension i is paired with i + rotary_dim / 2, the rotate-half convention;
     True: dimension 2i with 2i + 1; the frequencies are the same, and a mixer reads the flag: the
-    kernels that ``fused_rotary`` serves rotate halves, so a mixer must not hand them an interleaved part),
+    kernels that ``fused_rotary`` serves rotate halves, so a mixer hands them an interleaved part only after it
+    has put its query and key rows into ``half_order``),
     ignored_tensors (names below the mixer's prefix under which checkpoints of the family store
     a frequency table; it is computed here, so such a tensor is passed over)."""
     graph_safe = True
@@ -98,6 +103,13 @@ class Rotary(PositionEncoding):
 
     def load(self, tensors) -> None:
         pass
+
+    def half_order(self) -> List[int]:
+        """The order of a head's dimensions in which rotating halves is this part's rotation of pairs: the even
+        members of the rotated pairs, the odd ones, then the dimensions that do not rotate.  A score does not
+        change when query and key take one order, so a mixer may reorder the rows of its weights once."""
+        r = self.rotary_dim
+        return list(range(0, r, 2)) + list(range(1, r, 2)) + list(range(r, self.head_dim))
 
     def table(self, device) -> torch.Tensor:
         if self._table is None or self._table.device != device:

@@ -50,9 +50,24 @@ class PartSpec:
         raise KeyError(key)
 
 
+class FreeDim(int):
+    """A size that only the weight file gives (the rank of a low-rank pair, say).  As a number it is what the
+    random-weights mode draws; in a file any positive size is taken, the same one wherever the model's tensors
+    name ``key``."""
+
+    key: str
+
+    def __new__(cls, default: int, key: str) -> "FreeDim":
+        d = super().__new__(cls, default)
+        d.key = str(key)
+        return d
+
+
 @dataclass(frozen=True)
 class TensorSpec:
     """One tensor a part takes from the weight file.
+
+    shape: the sizes; a ``FreeDim`` among them is settled by the file.
 
     role: "matrix": held in the run's dtype (bfloat16 or float32);
           "vector": like a matrix, but a tensor that the file stores in 32-bit

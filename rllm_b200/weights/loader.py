@@ -27,7 +27,7 @@ from typing import Dict, Iterable, List, Optional, Sequence, Tuple
 
 import torch
 
-from ..parts.spec import TensorSpec
+from ..parts.spec import FreeDim, TensorSpec
 from .safetensors_io import SafetensorsFile, WeightsError, find_weight_files, write_safetensors
 
 class WeightsMismatch(WeightsError):
@@ -171,6 +171,21 @@ def _held_dtype(spec: TensorSpec, stored: torch.dtype, run_dtype: torch.dtype) -
     return run_dtype
 
 
+def _free_sizes(specs: Sequence[TensorSpec], source: WeightSource, have: Iterable[str]) -> Dict[str, int]:
+    """FreeDim key -> its size: what the first tensor that names it has in the file."""
+    have, sizes = set(have), {}
+    for s in specs:
+        if s.name not in have:
+            continue
+        shape = tuple(source.info(s.name)[1])
+        if len(shape) != len(s.shape):
+            continue
+        for want, got in zip(s.shape, shape):
+            if isinstance(want, FreeDim) and got > 0:
+                sizes.setdefault(want.key, int(got))
+    return sizes
+
+
 def check_tensors(specs: Sequence[TensorSpec], source: WeightSource, ignored: Iterable[str] = ()) -> None:
     """``ignored``: full names that the model's parts declared as present-but-unused."""
     have = set(source.names())
@@ -179,12 +194,14 @@ def check_tensors(specs: Sequence[TensorSpec], source: WeightSource, ignored: It
     missing = sorted(n for n, s in want.items() if n not in have and not s.optional)
     unexpected = sorted(n for n in have if n not in want and n not in skip)
     wrong_shape, wrong_kind = [], []
+    free = _free_sizes(specs, source, have)
     for n, s in want.items():
         if n not in have:
             continue
         dt, shape = source.info(n)
-        if tuple(shape) != tuple(s.shape):
-            wrong_shape.append((n, tuple(shape), tuple(s.shape)))
+        expected = tuple(free.get(d.key, int(d)) if isinstance(d, FreeDim) else d for d in s.shape)
+        if tuple(shape) != expected:
+            wrong_shape.append((n, tuple(shape), expected))
         if (s.role == "int") == dt.is_floating_point:
             wrong_kind.append((n, str(dt)))
     if missing or unexpected or wrong_shape or wrong_kind:
