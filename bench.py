@@ -514,6 +514,32 @@ TIBELIX_SIZES = {
 }
 
 
+def biranex(layers, width, dheads, ddim, dvdim, rank, heads, kv_heads, dim, window, sheads, sdim, state, groups, ff, vocab):
+    """layers of the pattern [gated delta rule, parallel (windowed attention beside a state-space recurrence) +
+    dense]: post-norm layers.  ``rank`` is not written: the random weights draw the low-rank pairs with the head's size."""
+    assert rank == ddim
+    delta = {"heads": dheads, "kv_heads": dheads, "dim": ddim, "vdim": dvdim, "conv": 4}
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                    "mask": {"size": window}, "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 4.0}}},
+           "left_scale": 0.9, "right_scale": 0.6,
+           "right": {"heads": sheads, "vdim": sdim, "state": state, "groups": groups, "conv": 4, "norm_groups": groups}}
+    return {"architecture": "Biranex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.8,
+            "max_positions": 8192,
+            "layers": [{"type": "channel_delta", "mixer": delta, "mlp": None} if i % 2 == 0 else
+                       {"type": "parallel", "mixer": par, "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+# Biranex beside Fevolorn (the closest design: linear-attention layers with a matrix state, and windowed attention
+# beside a state-space recurrence) of equal width, layers, vocabulary, attention and matrix-state sizes, and the
+# Llama of that width.  The state-space part has eight times Fevolorn's state a channel (128 against 16).
+BIRANEX_SIZES = {
+    "w1024": dict(layers=4, width=1024, dheads=8, ddim=64, dvdim=128, rank=64, heads=16, kv_heads=4, dim=64, window=512,
+                  sheads=32, sdim=64, state=128, groups=1, ff=2048, vocab=32768),
+    "w2048": dict(layers=4, width=2048, dheads=16, ddim=128, dvdim=128, rank=128, heads=16, kv_heads=4, dim=128,
+                  window=1024, sheads=64, sdim=64, state=128, groups=2, ff=4096, vocab=32768),
+}
+
+
 def compare_designs(args):
     """Prefill and decode throughput of Fasulix at sizes that resemble a real model's layers (random weights)
     beside the Llama of equal size, through the same step function; and, from one eager prefill step and one
@@ -593,6 +619,21 @@ def compare_designs(args):
             # q, k, v in, o out (float32), the gates; the state once in and once out per sequence
             return 4.0 * a[0].shape[0] * heads * d * dv, a[0].shape[0] * heads * (4.0 * d + 2.0 * dv + 4.0 * dv + 8.0) + \
                 8.0 * S * heads * (d * dv + d + 1)
+        if name == "postnorm_add":
+            terms = 1 if isinstance(a[1], torch.Tensor) else 2
+            return 0.0, a[0].numel() * (8.0 + 2.0 + 2.0 * terms)
+        if name == "ssd_scan":
+            heads, n, p = a[9], a[11], a[12]
+            # x, B, C and the steps in, y out (float32); the state once in and once out per sequence
+            return 4.0 * a[0].shape[0] * heads * n * p, 2.0 * a[0].numel() + 4.0 * a[0].shape[0] * heads * (p + 1) + \
+                8.0 * S * heads * n * p
+        if name == "silu_gated_group_rmsnorm":
+            return 0.0, 8.0 * a[0].numel()
+        if name in ("channel_delta_scan", "channel_delta_step"):
+            heads, d, dv = a[10], a[12], a[13]
+            # the convolutions' results, the decays' steps and beta in, o out (float32); the state in and out
+            return 6.0 * a[0].shape[0] * heads * d * dv, 2.0 * a[0].numel() + 4.0 * (a[1].numel() + a[2].numel()) + \
+                4.0 * a[0].shape[0] * heads * dv + 8.0 * S * heads * d * dv
         if name == "head_gated_rmsnorm":
             return 0.0, 8.0 * a[0].numel()
         if name in ("rms_mean2", "gated_rmsnorm"):
@@ -626,7 +667,8 @@ def compare_designs(args):
             "gemm_small_m_rstd", "gemm_tcgen05", "embedding", "lightning_scan", "selective_scan", "causal_conv",
             "streams_read", "streams_write", "head_norm_kv_write", "attention_simt_kv", "rms_mean2", "gated_rmsnorm",
             "act_mul", "moe_choose_sigmoid", "weighted_slot_sum", "layernorm", "add_rows", "add_row_bias", "mlstm_scan",
-            "head_gated_rmsnorm", "act", "sigmoid_gate")]
+            "head_gated_rmsnorm", "act", "sigmoid_gate", "postnorm_add", "ssd_scan", "silu_gated_group_rmsnorm",
+            "channel_delta_scan", "channel_delta_step", "activation_rows")]
         saved, log = {}, []
 
         def wrap(name, fn):
@@ -751,7 +793,10 @@ def compare_designs(args):
             row["fevolorn"] = measure("fevolorn", fevolorn(**FEVOLORN_SIZES[name]))
         if args.design == "tibelix":
             row["tibelix"] = measure("tibelix", tibelix(**TIBELIX_SIZES[name]))
-        if args.design == "munupel":
+        if args.design == "biranex":
+            row["biranex"] = measure("biranex", biranex(**BIRANEX_SIZES[name]))
+            row["fevolorn"] = measure("fevolorn", fevolorn(**FEVOLORN_SIZES[name]))
+        elif args.design == "munupel":
             row["munupel"] = measure("munupel", munupel(**MUNUPEL_SIZES[name]))
         else:
             row["fasulix"] = measure("fasulix", fasulix(**fx))
@@ -783,7 +828,7 @@ def main():
     ap.add_argument("--no-standin", action="store_true", help="skip the library-operator stand-in")
     ap.add_argument("--settle-steps", type=int, default=SETTLE_STEPS,
                     help="untimed decode steps of a device-timed point before its warm-up steps (0 for a short capture under a profiler)")
-    ap.add_argument("--design", default=None, choices=["fasulix", "fevolorn", "munupel", "tibelix"],
+    ap.add_argument("--design", default=None, choices=["biranex", "fasulix", "fevolorn", "munupel", "tibelix"],
                     help="instead of the default workload: this design beside the Llama of equal size (prefill and "
                          "decode throughput, kernels against their rooflines)")
     ap.add_argument("--design-size", default=None, help="only this entry of the design comparison's sizes")

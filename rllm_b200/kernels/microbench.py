@@ -10,6 +10,8 @@
     python -m rllm_b200.kernels.microbench lightning_scan --tokens 2048 --heads 16 --head-dim 128 --v-dim 128
     python -m rllm_b200.kernels.microbench selective_scan --tokens 2048 --channels 4096 --state 16
     python -m rllm_b200.kernels.microbench mlstm_scan --tokens 2048 --heads 8 --head-dim 128 --v-dim 256
+    python -m rllm_b200.kernels.microbench channel_delta --tokens 2048 --heads 16 --head-dim 128 --v-dim 128
+    python -m rllm_b200.kernels.microbench ssd_scan --tokens 2048 --heads 64 --head-dim 64 --state 128 --groups 1
     python -m rllm_b200.kernels.microbench streams --tokens 2048 --hidden 2048 --streams 4
 
 Sizes default to the Llama-3.2-1B shape (32 heads, 8 kv heads, head 64, hidden
@@ -303,6 +305,67 @@ def mlstm_scan(args) -> None:
           f"{moved / us / 1e3:.0f} GB/s of rows and state, {4.0 * T * heads * d * dv / us / 1e6:.2f} TFLOP/s float32")
 
 
+def channel_delta(args) -> None:
+    """The gated delta rule over one prompt portion, or one token of ``--batch`` sequences."""
+    heads, d, dv = args.heads, args.head_dim, args.v_dim or args.head_dim
+    q_start, _, slots, S, per = _one_sequence(args.tokens, args.batch)
+    T = S * per
+    bufs = [torch.randn(T, heads * (2 * d + dv), device=DEV).bfloat16() for _ in range(4)]
+    step, b = torch.randn(T, heads * d, device=DEV), torch.randn(T, heads, device=DEV)
+    dt_bias, a_log = torch.randn(heads * d, device=DEV) - 3, torch.randn(heads, device=DEV)
+    state = torch.zeros(S, heads, d, dv, device=DEV)
+    err = torch.zeros(1, dtype=torch.int32, device=DEV)
+
+    def run(i):
+        ops.channel_delta_scan(bufs[i % 4], step, b, dt_bias, a_log, 1e-6, state, q_start, slots, S, heads, heads, d, dv,
+                               err, max_q_len=per)
+    us = time_us(run, args.iters)
+    moved = T * heads * (4 * d + 2 * dv + 4 * d + 4 * dv + 4) + 8 * S * heads * d * dv
+    print(f"channel_delta tokens {T} ({S} sequences) heads {heads} x {d} x {dv}: {us:.1f} us, {moved / us / 1e3:.0f} GB/s "
+          f"of rows and state, {6.0 * T * heads * d * dv / us / 1e6:.2f} TFLOP/s of the recurrence")
+
+
+def channel_delta_step(args) -> None:
+    """One token of ``--batch`` sequences through the delta-rule layer's kernel, between its two products."""
+    heads, d, dv, H, r = args.heads, args.head_dim, args.v_dim or args.head_dim, args.hidden, 128
+    S, ch = args.batch, heads * (2 * d + dv)
+    bf = lambda *shape: (torch.randn(*shape, device=DEV) * 0.1).bfloat16()
+    a, x = bf(S, ch + 2 * r), bf(S, H)
+    w = {"b": bf(heads, H), "a2": bf(heads * d, r), "g2": bf(heads * dv, r), "conv": bf(ch, 4),
+         "dt_bias": torch.randn(heads * d, device=DEV) - 3, "a_log": torch.randn(heads, device=DEV),
+         "norm": torch.ones(heads * dv, device=DEV)}
+    n = max(1, (256 << 20) // (S * heads * d * dv * 4))             # states that together exceed L2
+    tails = torch.zeros(S, 3, ch, device=DEV)
+    states = [torch.zeros(S, heads, d, dv, device=DEV) for _ in range(n + 1)]
+    slots, err = torch.arange(S, dtype=torch.int32, device=DEV), torch.zeros(1, dtype=torch.int32, device=DEV)
+
+    def run(i):
+        ops.channel_delta_step(a, None, x, w, ch, ch + r, 4, 1e-6, 1e-6, tails, states[i % (n + 1)], slots, heads, heads,
+                               d, dv, err)
+    us = time_graph_us(run, args.iters)
+    print(f"channel_delta_step {S} sequences heads {heads} x {d} x {dv}: {us:.1f} us, "
+          f"{8 * S * heads * d * dv / us / 1e3:.0f} GB/s of state")
+
+
+def ssd_scan(args) -> None:
+    """The state-space recurrence over one prompt portion, or one token of ``--batch`` sequences."""
+    heads, p, n, groups = args.heads, args.head_dim, args.state, args.groups
+    q_start, _, slots, S, per = _one_sequence(args.tokens, args.batch)
+    T = S * per
+    bufs = [torch.randn(T, heads * p + 2 * groups * n, device=DEV).bfloat16() for _ in range(4)]
+    dt, vec = torch.randn(T, heads, device=DEV), lambda: torch.randn(heads, device=DEV)
+    dt_bias, a_log, skip = vec() - 3, vec(), vec()
+    state = torch.zeros(S, heads, n, p, device=DEV)
+    err = torch.zeros(1, dtype=torch.int32, device=DEV)
+
+    def run(i):
+        ops.ssd_scan(bufs[i % 4], dt, dt_bias, a_log, skip, state, q_start, slots, S, heads, groups, n, p, err, max_q_len=per)
+    us = time_us(run, args.iters)
+    moved = 2 * bufs[0].numel() + T * heads * (4 * p + 4) + 8 * S * heads * n * p
+    print(f"ssd_scan tokens {T} ({S} sequences) heads {heads} x {n} x {p}: {us:.1f} us, {moved / us / 1e3:.0f} GB/s "
+          f"of rows and state, {4.0 * T * heads * n * p / us / 1e6:.2f} TFLOP/s of the recurrence")
+
+
 def selective_scan(args) -> None:
     """The convolution and the selective recurrence over one prompt portion, or one token of ``--batch`` sequences."""
     E, N, R = args.channels, args.state, max(1, args.channels // 32)
@@ -349,7 +412,7 @@ def main(argv=None) -> int:
     p = argparse.ArgumentParser(prog="python -m rllm_b200.kernels.microbench", description=__doc__.split("\n\n")[0])
     p.add_argument("kernel", choices=["attention_decode", "attention_prefill", "gemm_small_m", "gemm_tcgen05",
                                       "latent_attention", "routed_experts", "lightning_scan", "selective_scan",
-                                      "streams", "mlstm_scan"])
+                                      "streams", "mlstm_scan", "channel_delta", "channel_delta_step", "ssd_scan"])
     p.add_argument("--batch", type=int, default=8)
     p.add_argument("--context", type=int, default=4096)
     p.add_argument("--tokens", type=int, default=2048)
@@ -373,7 +436,8 @@ def main(argv=None) -> int:
     p.add_argument("--gate", choices=["head", "element"], default=None, help="attention_*: a sigmoid gate on the result")
     p.add_argument("--v-dim", type=int, default=0, help="lightning_scan: a value head's size (0: --head-dim)")
     p.add_argument("--channels", type=int, default=4096, help="selective_scan: inner channels")
-    p.add_argument("--state", type=int, default=16, help="selective_scan: states a channel")
+    p.add_argument("--state", type=int, default=16, help="selective_scan: states a channel; ssd_scan: states a head's column")
+    p.add_argument("--groups", type=int, default=1, help="ssd_scan: groups of heads that share B and C")
     p.add_argument("--streams", type=int, default=4, help="streams: residual streams")
     p.add_argument("--experts", type=int, default=32)
     p.add_argument("--top", type=int, default=4)
@@ -390,7 +454,9 @@ def main(argv=None) -> int:
     {"attention_decode": attention_decode, "attention_prefill": attention_prefill,
      "gemm_small_m": gemm_small_m, "gemm_tcgen05": gemm_tcgen05, "latent_attention": latent_attention,
      "routed_experts": routed_experts, "lightning_scan": lightning_scan, "selective_scan": selective_scan,
-     "streams": streams, "mlstm_scan": mlstm_scan}[args.kernel](args)
+     "streams": streams, "mlstm_scan": mlstm_scan, "channel_delta": channel_delta,
+     "channel_delta_step": channel_delta_step,
+     "ssd_scan": ssd_scan}[args.kernel](args)
     return 0
 
 

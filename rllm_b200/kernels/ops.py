@@ -1560,15 +1560,21 @@ def silu_gated_group_rmsnorm(y: torch.Tensor, z: torch.Tensor, weight: torch.Ten
 # ---------------------------------------------------------------------------
 # the gated delta rule with a decay per key channel (channel_delta.cu)
 # ---------------------------------------------------------------------------
+CHANNEL_DELTA_CHUNKED_FROM = 16        # longest portion from which bfloat16 steps go sixteen tokens at a time
+CHANNEL_DELTA_WORK_BYTES = 64 << 20
+
+
 def channel_delta_scan(c: torch.Tensor, step: torch.Tensor, b: torch.Tensor, dt_bias: torch.Tensor,
                        a_log: torch.Tensor, unit_eps: float, state: torch.Tensor, q_start: torch.Tensor,
                        slots: torch.Tensor, num_seqs: int, heads: int, kv: int, d: int, dv: int,
-                       err: torch.Tensor) -> torch.Tensor:
+                       err: torch.Tensor, max_q_len: int = 1) -> torch.Tensor:
     """The delta rule over this step's tokens of every sequence, in order, from and into the sequences' slots.
     c [T, 2 kv d + heads dv]: q | k | v after their convolutions; step float32 [T, heads d]: the decays' step
     before bias and softplus; b float32 [T, heads]: beta before its sigmoid; dt_bias float32 [heads d], a_log
     float32 [heads]; state float32 [slots, heads, d, dv].  q and k are made unit vectors (``unit_eps`` under the
-    root), q is multiplied by d^(-1/2).  Returns o float32 [T, heads dv]."""
+    root), q is multiplied by d^(-1/2).  Returns o float32 [T, heads dv].  Portions of bfloat16 activations take the
+    tensor-core form, sixteen tokens at a time (d up to 128); the result differs by rounding only."""
+    import os
     lib = build.load_library("channel_delta")
     T = c.shape[0]
     assert c.shape[1] == 2 * kv * d + heads * dv and c.stride(1) == 1
@@ -1579,10 +1585,28 @@ def channel_delta_scan(c: torch.Tensor, step: torch.Tensor, b: torch.Tensor, dt_
     assert state.dtype is torch.float32 and tuple(state.shape[1:]) == (heads, d, dv)
     for t, name in ((step, "step"), (b, "b"), (dt_bias, "dt_bias"), (a_log, "a_log"), (state, "state")):
         _contig(t, name)
+    stride = c.stride(0) if T > 1 else c.shape[1]
     f32 = dict(dtype=torch.float32, device=c.device)
+    if c.dtype is torch.bfloat16 and max_q_len >= CHANNEL_DELTA_CHUNKED_FROM and \
+            os.environ.get("RLLM_CHANNEL_DELTA") != "simt":
+        per = int(lib.rllm_channel_delta_chunk_bytes(c_int(d), c_int(dv))) * num_seqs * heads
+        chunks = -(-max_q_len // 16)
+        # the records of a call stay in L2: as many chunks at a time as fit, in equal parts
+        calls = max(1, -(-chunks * per // CHANNEL_DELTA_WORK_BYTES), -(-chunks * num_seqs // 65535))
+        seg = -(-chunks // min(calls, chunks))
+        if per and seg * num_seqs <= 65535:
+            out = torch.empty((T, heads * dv), **f32)
+            work = torch.empty(seg * per, dtype=torch.uint8, device=c.device)
+            for chunk0 in range(0, chunks, seg):
+                _check(lib.rllm_channel_delta_chunked(_ptr(c), c_int(stride), _ptr(step), _ptr(b), _ptr(dt_bias),
+                                                      _ptr(a_log), c_float(unit_eps), c_float(float(d) ** -0.5),
+                                                      _ptr(state), _ptr(q_start), _ptr(slots), c_int(state.shape[0]),
+                                                      c_int(num_seqs), c_int(chunk0), c_int(seg), _ptr(work), _ptr(out),
+                                                      c_int(heads), c_int(kv), c_int(d), c_int(dv), _ptr(err),
+                                                      _stream()), "channel_delta_chunked")
+            return out
     qn, kn, g = torch.empty((T, kv, d), **f32), torch.empty((T, kv, d), **f32), torch.empty((T, heads, d), **f32)
     beta, out = torch.empty((T, heads), **f32), torch.empty((T, heads * dv), **f32)
-    stride = c.stride(0) if T > 1 else c.shape[1]
     _check(lib.rllm_channel_delta_prepare(_ptr(c), c_int(stride), c_int(dtype_code(c.dtype)), _ptr(step), _ptr(b),
                                           _ptr(dt_bias), _ptr(a_log), _ptr(qn), _ptr(kn), _ptr(g), _ptr(beta), c_int(T),
                                           c_int(heads), c_int(kv), c_int(d), c_float(unit_eps),
@@ -1592,4 +1616,50 @@ def channel_delta_scan(c: torch.Tensor, step: torch.Tensor, b: torch.Tensor, dt_
                                        c_int(dtype_code(c.dtype)), _ptr(state), _ptr(q_start), _ptr(slots),
                                        c_int(state.shape[0]), c_int(num_seqs), _ptr(out), c_int(heads), c_int(kv),
                                        c_int(d), c_int(dv), _ptr(err), _stream()), "channel_delta_walk")
+    return out
+
+
+def channel_delta_step_takes(d: int, dv: int, rank_a: int, rank_g: int) -> bool:
+    """Whether ``channel_delta_step`` takes these sizes (heads up to 128 x 256, whole groups of four value columns)."""
+    lib = build.load_library("channel_delta")
+    return bool(lib.rllm_channel_delta_step_takes(c_int(d), c_int(dv), c_int(rank_a), c_int(rank_g)))
+
+
+def channel_delta_step(a: torch.Tensor, c: Optional[torch.Tensor], x: torch.Tensor, w, at_a: int, at_g: int,
+                       taps: int, unit_eps: float, eps: float, tail: torch.Tensor, state: torch.Tensor,
+                       slots: torch.Tensor, heads: int, kv: int, d: int, dv: int, err: torch.Tensor,
+                       early: bool = False) -> torch.Tensor:
+    """One token of every sequence through the delta rule, from the mixer's first product to its output product's
+    input.  a [S, .]: q | k | v (before their convolutions), W_a1 h from column ``at_a``, W_g1 h from ``at_g``; c
+    [S, 2 kv d + heads dv]: the convolutions' results, or None where ``kv == heads`` (they are then made here, from
+    and into ``tail`` float32 [slots, taps - 1, channels]); x [S, H]: the mixer's input; w: the tensors b [heads, H],
+    a2 [heads d, rank], g2 [heads dv, rank] (ranks multiples of 8), conv [channels, taps], and float32 dt_bias, a_log,
+    norm [>= dv]; state float32 [slots, heads, d, dv], updated in place.  ``early``: the kernel launched directly ahead
+    does not write ``state``, so that it may be fetched while that one still runs.  Returns the gated, normalised result
+    [S, heads dv] in a's dtype."""
+    lib = build.load_library("channel_delta")
+    S, ch = a.shape[0], 2 * kv * d + heads * dv
+    assert a.stride(1) == 1 and x.shape[0] == S and x.stride(1) == 1 and x.dtype is a.dtype
+    ra, rg = w["a2"].shape[1], w["g2"].shape[1]
+    for k in ("b", "a2", "g2"):
+        assert w[k].dtype is a.dtype
+        _contig(w[k], k)
+    assert w["a2"].shape[0] == heads * d and w["g2"].shape[0] == heads * dv and w["b"].shape == (heads, x.shape[1])
+    assert w["a2"].data_ptr() % 16 == 0 and w["g2"].data_ptr() % 16 == 0
+    assert w["conv"].shape == (ch, taps) and w["conv"].is_contiguous()
+    assert at_a + ra <= a.shape[1] and at_g + rg <= a.shape[1]
+    for k in ("dt_bias", "a_log", "norm"):
+        assert w[k].dtype is torch.float32
+    assert state.dtype is torch.float32 and tuple(state.shape[1:]) == (heads, d, dv) and state.is_contiguous()
+    assert tail.dtype is torch.float32 and tuple(tail.shape[1:]) == (taps - 1, ch) and tail.is_contiguous()
+    if c is not None:
+        assert c.shape == (S, ch) and c.dtype is a.dtype and c.is_contiguous()
+    out = torch.empty((S, heads * dv), dtype=a.dtype, device=a.device)
+    _check(lib.rllm_channel_delta_step(
+        _ptr(a), c_int(a.stride(0)), _ptr(c), _ptr(x), c_int(x.stride(0)), _ptr(w["b"]), _ptr(w["a2"]), _ptr(w["g2"]),
+        _ptr(w["conv"]), c_int(dtype_code(w["conv"].dtype)), _ptr(w["dt_bias"]), _ptr(w["a_log"]), _ptr(w["norm"]),
+        _ptr(tail), _ptr(state), _ptr(slots), _ptr(out), c_int(dtype_code(a.dtype)), c_int(S), c_int(at_a), c_int(at_g),
+        c_int(ra), c_int(rg), c_int(x.shape[1]), c_int(taps), c_int(state.shape[0]), c_int(heads), c_int(kv), c_int(d),
+        c_int(dv), c_float(unit_eps), c_float(float(d) ** -0.5), c_float(eps), c_int(1 if early else 0), _ptr(err),
+        _stream()), "channel_delta_step")
     return out

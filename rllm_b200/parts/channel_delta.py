@@ -11,7 +11,8 @@ Per request the part keeps two states, both float32: S [heads, d, dv] and the co
 inputs ([taps - 1, 2 kv_heads d + heads dv]); both start at zero.  q, k, v and the low-rank inputs W_a1 h,
 W_g1 h are one matrix product over the stacked weights; beta's and the decays' pre-activations are products
 whose results stay float32; unit vectors, logarithms, exponentials, the recurrence and the norm are float32
-arithmetic in the kernels.  The ranks of the two low-rank pairs are the tensors' own.
+arithmetic in the kernels.  Steps in which every sequence brings one token take one kernel between the first
+and the last product (``ops.channel_delta_step``).  The ranks of the two low-rank pairs are the tensors' own.
 
 params: hidden_size, num_heads, num_kv_heads, head_dim, v_dim, conv (taps), eps, unit_eps, rank (optional: what
 the random-weights mode draws; head_dim if absent), tensor_names (keys "q", "k", "v", "q_conv", "k_conv",
@@ -19,7 +20,8 @@ the random-weights mode draws; head_dim if absent), tensor_names (keys "q", "k",
 """
 from __future__ import annotations
 
-from typing import Dict, List, Optional
+import os
+from typing import Dict, List
 
 import torch
 
@@ -94,20 +96,34 @@ class ChannelDelta(Mixer):
                   # what enters float32 arithmetic is kept so, whatever the run's dtype
                   "a_log": t["a_log"].float().contiguous(), "dt_bias": t["dt_bias"].float().contiguous(),
                   "norm": t["norm"].float().repeat(self.heads).contiguous()}
+        self.step_kernel = t["o"].is_cuda and os.environ.get("RLLM_CHANNEL_DELTA") != "simt" and \
+            ops.channel_delta_step_takes(self.d, self.dv, self.w["a2"].shape[1], self.w["g2"].shape[1])
 
     def cache_need(self):
         return (StateNeed((self.heads, self.d, self.dv)), StateNeed((self.taps - 1, self.channels)))
+
+    def _conv(self, a: torch.Tensor, tail, ctx: StepContext) -> torch.Tensor:
+        return ops.causal_conv(a[:, :self.channels], self.w["conv"], None, tail.state, ctx.q_start, ctx.token_seq,
+                               ctx.state_slots, ctx.num_seqs, ctx.num_tokens > ctx.num_decode, ctx.err)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache) -> torch.Tensor:
         memory, tail = cache
         w = self.w
         a = linear(x, w["in"])                                               # q | k | v | W_a1 h | W_g1 h
+        if ctx.num_tokens == ctx.num_decode and self.step_kernel:
+            # decoding: everything up to the output product in one kernel (the convolutions too, unless heads
+            # share a q/k head, whose last inputs then have one writer: the convolution's own kernel)
+            c = None if self.kv == self.heads else self._conv(a, tail, ctx)
+            y = ops.channel_delta_step(a, c, x, w, self.at_a, self.at_g, self.taps, self.unit_eps, self.eps,
+                                       tail.state, memory.state, ctx.state_slots, self.heads, self.kv, self.d, self.dv,
+                                       ctx.err, early=True)
+            return linear(y, w["o"])
         b = linear(x, w["b"], out_dtype=torch.float32)                       # [T, heads]
-        c = ops.causal_conv(a[:, :self.channels], w["conv"], None, tail.state, ctx.q_start, ctx.token_seq,
-                            ctx.state_slots, ctx.num_seqs, ctx.num_tokens > ctx.num_decode, ctx.err)
+        c = self._conv(a, tail, ctx)
         step = linear(a[:, self.at_a:self.at_g], w["a2"], out_dtype=torch.float32)     # [T, heads d]
         gate = linear(a[:, self.at_g:self.end_g], w["g2"])                             # [T, heads dv]
         o = ops.channel_delta_scan(c, step, b, w["dt_bias"], w["a_log"], self.unit_eps, memory.state, ctx.q_start,
-                                   ctx.state_slots, ctx.num_seqs, self.heads, self.kv, self.d, self.dv, ctx.err)
+                                   ctx.state_slots, ctx.num_seqs, self.heads, self.kv, self.d, self.dv, ctx.err,
+                                   max_q_len=ctx.max_q_len)
         y = ops.head_gated_rmsnorm(o, gate, w["norm"], self.eps, self.heads, x.dtype)
         return linear(y, w["o"])
