@@ -457,9 +457,9 @@ RLLM_EXPORT int rllm_channel_delta_chunked(const void* c, int c_stride, const fl
     rllm_launch_pdl(channel_delta_records_kernel<D_>, dim3(heads, num_seqs * seg), dim3(CDM_PREP_THREADS), (size_t)0, \
                     stream, (const bf16*)c, c_stride, step, b, dt_bias, a_log, q_start, chunk0, seg, rec, u0, heads, \
                     kv, d, dv, dvp, unit_eps, qscale);                                                               \
-    const size_t smem = CDM_STAGES * sizeof(CdmRecord<D_>) + 4 * 4 * 32 * sizeof(float4);                            \
+    const size_t smem = sizeof(CdmSmem<D_>);                                                                         \
     cudaFuncSetAttribute(channel_delta_chunks_kernel<D_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
-    rllm_launch_pdl(channel_delta_chunks_kernel<D_>, dim3(dvp / 16, heads, num_seqs), dim3(128), smem, stream,       \
+    rllm_launch_pdl(channel_delta_chunks_kernel<D_>, dim3(dvp / 16, heads, num_seqs), dim3(CDM_THREADS), smem, stream, \
                     (const CdmRecord<D_>*)rec, (const float*)u0, state, q_start, slots, num_slots, chunk0, seg, out, \
                     heads, d, dv, dvp, err);                                                                         \
   } while (0)
