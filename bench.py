@@ -629,7 +629,11 @@ def compare_designs(args):
                 8.0 * S * heads * n * p
         if name == "silu_gated_group_rmsnorm":
             return 0.0, 8.0 * a[0].numel()
-        if name in ("channel_delta_scan", "channel_delta_step"):
+        if name == "channel_delta_step":
+            heads, d, dv = a[12], a[14], a[15]
+            # the second low-rank products' weights and beta's, the token's rows; the state in and out
+            return 0.0, 2.0 * (a[0].numel() + sum(a[3][k].numel() for k in ("b", "a2", "g2"))) + 8.0 * S * heads * d * dv
+        if name == "channel_delta_scan":
             heads, d, dv = a[10], a[12], a[13]
             # the convolutions' results, the decays' steps and beta in, o out (float32); the state in and out
             return 6.0 * a[0].shape[0] * heads * d * dv, 2.0 * a[0].numel() + 4.0 * (a[1].numel() + a[2].numel()) + \
