@@ -458,10 +458,14 @@ RLLM_EXPORT int rllm_channel_delta_chunked(const void* c, int c_stride, const fl
                     stream, (const bf16*)c, c_stride, step, b, dt_bias, a_log, q_start, chunk0, seg, rec, u0, heads, \
                     kv, d, dv, dvp, unit_eps, qscale);                                                               \
     const size_t smem = sizeof(CdmSmem<D_>);                                                                         \
-    cudaFuncSetAttribute(channel_delta_chunks_kernel<D_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);   \
-    rllm_launch_pdl(channel_delta_chunks_kernel<D_>, dim3(dvp / 16, heads, num_seqs), dim3(CDM_THREADS), smem, stream, \
-                    (const CdmRecord<D_>*)rec, (const float*)u0, state, q_start, slots, num_slots, chunk0, seg, out, \
-                    heads, d, dv, dvp, err);                                                                         \
+    static bool allowed = false;                                                                                     \
+    if (!allowed) {                                                                                                  \
+      cudaFuncSetAttribute(channel_delta_chunks_kernel<D_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+      allowed = true;                                                                                                \
+    }                                                                                                                \
+    /* an ordinary launch: blocks that came in early, as records' blocks leave, would share SMs while others idle */  \
+    channel_delta_chunks_kernel<D_><<<dim3(dvp / 16, heads, num_seqs), dim3(CDM_THREADS), smem, stream>>>(           \
+        rec, u0, state, q_start, slots, num_slots, chunk0, seg, out, heads, d, dv, dvp, err);                        \
   } while (0)
   if (cdm_size(d) == 64) CDM_GO(64); else CDM_GO(128);
 #undef CDM_GO

@@ -7,7 +7,7 @@ rotated dims at a third of their frequency and a window of 11 (shorter than a pa
 9 taps and a feed-forward; a second parallel layer without a feed-forward, with a window over several pages.
 BX_B: multiples of 16: the sizes of the tensor-core kernels (attention heads of 64 and 128 with keys and values of
 one size, delta heads of 64 x 128 and 128 x 64, state-space heads of 64 x 64 and 128 x 32).
-BX_C: values that make mechanisms trivial: one head, one tap, a window of one token, nothing rotated but one pair and
+BX_C: a width that is no multiple of 8, and values that make mechanisms trivial: one head, one tap, a window of one token, nothing rotated but one pair and
 no rescaling, a left scale of zero, a group a head; keys of 32 and values of 16 (rows of one size in the pages).
 """
 from __future__ import annotations
@@ -55,7 +55,7 @@ BX_B = {
     ],
 }
 BX_C = {
-    "architecture": "Biranex", "vocab": 97, "width": 40, "norm": {"eps": 1e-3}, "residual_mult": 1.0,
+    "architecture": "Biranex", "vocab": 97, "width": 45, "norm": {"eps": 1e-3}, "residual_mult": 1.0,
     "layers": [
         layer(par((1, 1, 8, 12, 0.4, 1, 50.0, 2, None), 1.0, (1, 24, 1, 1, 1, 1), 1.0), 24),
         layer(delta(1, 1, 8, 4, 1)),
