@@ -59,13 +59,16 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
                       int nq, int nkv, int d, int dv, int page_size, int num_pages, int window, float scale,
                       int keep_first, int chunk, float softcap, const float* __restrict__ sinks,
                       const T* __restrict__ gate, int gate_stride, int gate_mode,
-                      const float* __restrict__ slopes, int* __restrict__ err) {
+                      const float* __restrict__ slopes, int shared_keys, int v_ld, int* __restrict__ err) {
   extern __shared__ float qs[];  // [ATT_WARPS][d]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const long long gw = (long long)blockIdx.x * ATT_WARPS + warp;
   if (gw >= (long long)T_tokens * nq) return;
   const int t = (int)(gw / nq), h = (int)(gw - (long long)t * nq);
   const int kvh = h / (nq / nkv);
+  // rows of the caches: which head of a page, how many heads it has, and where a value row of it starts
+  const int pg_heads = shared_keys ? 1 : nkv, pg_h = shared_keys ? 0 : kvh;
+  const int v_row = shared_keys ? nkv * v_ld : dv, v_off = shared_keys ? kvh * v_ld : 0;
   const int s = token_seq[t];
   const int qpos = positions[t];
   const int kend = qpos + 1;
@@ -100,7 +103,7 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
         atomicOr(err, 4);
         page = -1;
       } else {
-        const T* kp = kcache + (((size_t)page * nkv + kvh) * page_size + (j % page_size)) * d;
+        const T* kp = kcache + (((size_t)page * pg_heads + pg_h) * page_size + (j % page_size)) * d;
         float dot = 0.f;
         if (VEC) {
           for (int i = 0; i < d; i += 8) {
@@ -131,7 +134,7 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       const int pg = __shfl_sync(0xffffffffu, page, jj);
       if (pg < 0) continue;
-      const T* vp = vcache + (((size_t)pg * nkv + kvh) * page_size + ((j0 + jj) % page_size)) * dv;
+      const T* vp = vcache + (((size_t)pg * pg_heads + pg_h) * page_size + ((j0 + jj) % page_size)) * v_row + v_off;
 #pragma unroll
       for (int r = 0; r < ATT_MAX_D / 32; ++r) {
         const int i = lane + 32 * r;
@@ -163,20 +166,21 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out
   }
 }
 
-// keys [pages, nkv, page_size, d], values [pages, nkv, page_size, dv], out [T, nq * dv]
+// keys [pages, nkv, page_size, d], values [pages, nkv, page_size, dv], out [T, nq * dv]; with shared_keys: keys
+// [pages, 1, page_size, d], values [pages, 1, page_size, nkv * v_ld]
 RLLM_EXPORT int rllm_attention_simt_kv(const void* q, int q_stride, void* out, const void* kcache,
                                        const void* vcache, int dtype, const int* block_table,
                                        int max_blocks, const int* positions, const int* token_seq, int T,
                                        int nq, int nkv, int d, int dv, int page_size, int num_pages, int window,
                                        float scale, int keep_first, int chunk, float softcap, const float* sinks,
                                        const void* gate, int gate_stride, int gate_mode, const float* slopes,
-                                       int* err, cudaStream_t stream) {
+                                       int shared_keys, int v_ld, int* err, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (nq <= 0 || nkv <= 0 || nq % nkv != 0 || d <= 0 || dv <= 0 || page_size <= 0 || num_pages <= 0 ||
       max_blocks <= 0 || window < 0 || keep_first < 0 || chunk < 0 || !(softcap >= 0.f) || gate_mode < 0 ||
-      gate_mode > 2 || (gate_mode && !gate))
+      gate_mode > 2 || (gate_mode && !gate) || (shared_keys && v_ld < dv))
     return RLLM_E_BADARG;
-  if (dv > ATT_MAX_D || d > 1024) return RLLM_E_UNSUPPORTED;
+  if (dv > ATT_MAX_D || d > 2816) return RLLM_E_UNSUPPORTED;
   const bool vec = d % 8 == 0 && q_stride % 8 == 0 && (((uintptr_t)q | (uintptr_t)kcache) & 31) == 0;
   const long long warps = (long long)T * nq;
   const unsigned blocks = (unsigned)((warps + ATT_WARPS - 1) / ATT_WARPS);
@@ -186,7 +190,7 @@ RLLM_EXPORT int rllm_attention_simt_kv(const void* q, int q_stride, void* out, c
     (attention_simt_kernel<T_, VEC_><<<blocks, 32 * ATT_WARPS, smem, stream>>>(                             \
         (const T_*)q, q_stride, (T_*)out, (const T_*)kcache, (const T_*)vcache, block_table,                \
         max_blocks, positions, token_seq, T, nq, nkv, d, dv, page_size, num_pages, window, scale, keep_first,  \
-        chunk, softcap, sinks, (const T_*)gate, gate_stride, gate_mode, slopes, err)))
+        chunk, softcap, sinks, (const T_*)gate, gate_stride, gate_mode, slopes, shared_keys, v_ld, err)))
   if (vec) ATT_GO(true); else ATT_GO(false);
 #undef ATT_GO
   RLLM_LAUNCH_CHECK();
@@ -202,5 +206,5 @@ RLLM_EXPORT int rllm_attention_simt(const void* q, int q_stride, void* out, cons
   if (q_stride % 8 != 0) return RLLM_E_BADARG;
   return rllm_attention_simt_kv(q, q_stride, out, kcache, vcache, dtype, block_table, max_blocks, positions,
                                 token_seq, T, nq, nkv, d, d, page_size, num_pages, window, scale, 0, 0, 0.f, nullptr,
-                                nullptr, 0, 0, nullptr, err, stream);
+                                nullptr, 0, 0, nullptr, 0, 0, err, stream);
 }

@@ -56,6 +56,15 @@ __device__ __forceinline__ float block_sum(float v, float* smem32) {
   return t;
 }
 
+// The gate of a gated feed-forward: g' sigmoid(slope g') (u' + shift) with g' = min(g, limit) and u' = u kept within
+// +-limit.  {infinity, 1, 0}: silu(g) u.
+struct GateAct { float limit, slope, shift; };
+__device__ __forceinline__ float gate_act(float g, float u, const GateAct& p) {
+  g = fminf(g, p.limit);
+  u = fminf(fmaxf(u, -p.limit), p.limit);
+  return g / (1.0f + expf(-p.slope * g)) * (u + p.shift);
+}
+
 // cos and sin of position * inv_freq for the bfloat16 path: the angle is reduced
 // mod 2 pi in float64 (exact to ~1e-11 for positions up to 2^20), then cosine
 // and sine are taken in float32 (absolute error ~2e-7).  The float32 path of the

@@ -385,22 +385,23 @@ RLLM_EXPORT int rllm_rope_kv_write(void* qkv, int dtype, const int* positions, c
 }
 
 // ---------------------------------------------------------------------------
-// out[t, i] = silu(gu[t, i]) * gu[t, I + i],  silu(z) = z / (1 + exp(-z))
+// out[t, i] = silu(gu[t, i]) * gu[t, I + i],  silu(z) = z / (1 + exp(-z)), with the gate's constants of GateAct
 // (crates/rllm-model/src/layers.rs:214-220), float32 arithmetic.
 // ---------------------------------------------------------------------------
 template <typename T>
-__global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, size_t n) {
+__global__ void silu_mul_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, size_t n, GateAct ga) {
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n) return;
   const size_t t = idx / I;
   const int i = (int)(idx - t * I);
   const float g = to_f32(gu[t * 2 * I + i]);
   const float u = to_f32(gu[t * 2 * I + I + i]);
-  out[idx] = from_f32<T>(g / (1.0f + expf(-g)) * u);
+  out[idx] = from_f32<T>(gate_act(g, u, ga));
 }
 
 // bfloat16 with I a multiple of 8: 16-byte loads and stores, 8 values a thread
-__global__ void silu_mul_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, int I8, size_t n8) {
+__global__ void silu_mul_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __restrict__ out, int I8, size_t n8,
+                                       GateAct ga) {
   size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= n8) return;
   const size_t t = idx / I8;
@@ -414,7 +415,7 @@ __global__ void silu_mul_bf16x8_kernel(const bf16* __restrict__ gu, bf16* __rest
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const float2 gf = __bfloat1622float2(gp[k]), uf = __bfloat1622float2(up[k]);
-    op[k] = __floats2bfloat162_rn(gf.x / (1.0f + expf(-gf.x)) * uf.x, gf.y / (1.0f + expf(-gf.y)) * uf.y);
+    op[k] = __floats2bfloat162_rn(gate_act(gf.x, uf.x, ga), gate_act(gf.y, uf.y, ga));
   }
   *(uint4*)(out + idx * 8) = o;
 }
@@ -490,19 +491,22 @@ RLLM_EXPORT int rllm_sigmoid_gate(const void* x, const void* g, int g_stride, vo
   return 0;
 }
 
-RLLM_EXPORT int rllm_silu_mul(const void* gu, void* out, int dtype, int T, int I, cudaStream_t stream) {
+// limit, slope, shift: the gate's constants (GateAct)
+RLLM_EXPORT int rllm_silu_mul(const void* gu, void* out, int dtype, int T, int I, float limit, float slope, float shift,
+                              cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (I <= 0) return RLLM_E_BADARG;
+  if (I <= 0 || !(limit > 0.f)) return RLLM_E_BADARG;
+  const GateAct ga{limit, slope, shift};
   if (dtype == RLLM_DT_BF16 && I % 8 == 0 && (((uintptr_t)gu | (uintptr_t)out) & 15) == 0) {
     const size_t n8 = (size_t)T * (I / 8);
-    silu_mul_bf16x8_kernel<<<(unsigned)((n8 + 255) / 256), 256, 0, stream>>>((const bf16*)gu, (bf16*)out, I / 8, n8);
+    silu_mul_bf16x8_kernel<<<(unsigned)((n8 + 255) / 256), 256, 0, stream>>>((const bf16*)gu, (bf16*)out, I / 8, n8, ga);
     RLLM_LAUNCH_CHECK();
     return 0;
   }
   size_t n = (size_t)T * I;
   unsigned blocks = (unsigned)((n + 255) / 256);
   RLLM_DISPATCH_DTYPE(dtype, T_,
-    (silu_mul_kernel<T_><<<blocks, 256, 0, stream>>>((const T_*)gu, (T_*)out, I, n)));
+    (silu_mul_kernel<T_><<<blocks, 256, 0, stream>>>((const T_*)gu, (T_*)out, I, n, ga)));
   RLLM_LAUNCH_CHECK();
   return 0;
 }
@@ -531,4 +535,26 @@ RLLM_EXPORT int rllm_decode_advance(int* token_ids, int* positions, int* seq_len
   if (S <= 0) return 0;
   return (int)rllm_launch_pdl(decode_advance_kernel, dim3((S + 127) / 128), dim3(128), 0, stream, token_ids, positions,
                               seq_lens, sampled, history_row, S);
+}
+
+// ---------------------------------------------------------------------------
+// x <- cap * tanh(x / cap), element by element (logits)
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) softcap_kernel(float* x, long long n, float cap) {
+  pdl_wait_on(x);
+  pdl_launch();
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (i + 4 <= n && (((uintptr_t)x) & 15) == 0) {
+    float4 v = *(float4*)(x + i);
+    v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+    *(float4*)(x + i) = v;
+  } else {
+    for (long long j = i; j < n && j < i + 4; ++j) x[j] = cap * tanhf(x[j] / cap);
+  }
+}
+
+RLLM_EXPORT int rllm_softcap(float* x, long long n, float cap, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (!(cap > 0.f)) return RLLM_E_BADARG;
+  return (int)rllm_launch_pdl(softcap_kernel, dim3((unsigned)((n + 1023) / 1024)), dim3(256), (size_t)0, stream, x, n, cap);
 }

@@ -26,6 +26,7 @@
 // adds up a row's partial sums in a fixed order and multiplies row m of its
 // result by 1 / sqrt(mean(h[m]^2) + eps).
 #include "common.cuh"
+#include <math.h>
 #include <stdlib.h>
 
 #define EPI_BF16 0
@@ -59,6 +60,8 @@ struct NormSide {
   float* parts_out;                                     // out: [gridDim.x, M]
   const void* w_next; int w_is_f32;                     // out: weight [N] of the norm that reads h next (or null)
   bf16* scaled; int lds;                                // out: [M, N] = bfloat16(h * w_next)
+  GateAct ga;                                           // the SiLU-gate epilogue's constants
+  const float* alpha; const void* shift;                // out: with alpha [1], scaled = bfloat16(tanh(alpha h) w_next + shift)
 };
 
 // The parts of row m = tid % R (R = 8 MT rows) that fall to this thread's slice tid / R, added in order; the
@@ -218,7 +221,9 @@ gemm_small_m_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
         *hp = hv;
         if (ns.scaled) {
           const float wv = ns.w_is_f32 ? ((const float*)ns.w_next)[n] : __bfloat162float(((const bf16*)ns.w_next)[n]);
-          ns.scaled[(size_t)m * ns.lds + n] = __float2bfloat16_rn(hv * wv);
+          float sv = hv * wv;
+          if (ns.alpha) sv = fmaf(tanhf(ns.alpha[0] * hv), wv, ns.w_is_f32 ? ((const float*)ns.shift)[n] : __bfloat162float(((const bf16*)ns.shift)[n]));
+          ns.scaled[(size_t)m * ns.lds + n] = __float2bfloat16_rn(sv);
         }
       }
       tile[m * 16 + r] = hv;
@@ -240,7 +245,7 @@ gemm_small_m_kernel(const bf16* __restrict__ x, int ldx, const bf16* __restrict_
       }
       const int n = n0 + r;
       if (RSTD) { g *= s_rstd[m]; u *= s_rstd[m]; }
-      if (m < M && n < N) ((bf16*)out)[(size_t)m * ldo + n] = __float2bfloat16_rn(g / (1.0f + expf(-g)) * u);
+      if (m < M && n < N) ((bf16*)out)[(size_t)m * ldo + n] = __float2bfloat16_rn(gate_act(g, u, ns.ga));
     }
   } else {
     for (int idx = threadIdx.x; idx < 16 * cols; idx += blockDim.x) {
@@ -317,17 +322,19 @@ static int launch_small_m(const bf16* x, int ldx, const bf16* W, int ldw, void* 
 
 template <int EPI>
 static int dispatch_mt(const bf16* x, int ldx, const bf16* W, int ldw, void* out, int ldo, int M, int N, int K,
-                       int up_offset, cudaStream_t stream) {
+                       int up_offset, cudaStream_t stream, GateAct ga = GateAct{INFINITY, 1.f, 0.f}) {
   NormSide none = {};
+  none.ga = ga;
   if (M <= 8) return launch_small_m<1, EPI, false>(x, ldx, W, ldw, out, ldo, M, N, K, up_offset, none, stream);
   if (M <= 16) return launch_small_m<2, EPI, false>(x, ldx, W, ldw, out, ldo, M, N, K, up_offset, none, stream);
   return RLLM_E_UNSUPPORTED;
 }
 
 // epilogue 0: out bfloat16 [M, N]; 1: out float32 [M, N]; 2: W = [gate rows (N); up rows (N)] stacked
-// (2 N rows in all), out bfloat16 [M, N] = silu(x . gate^T) * (x . up^T).
+// (2 N rows in all), out bfloat16 [M, N] = silu(x . gate^T) * (x . up^T), with the gate's constants (GateAct).
 RLLM_EXPORT int rllm_gemm_small_m(const void* x, int ldx, const void* W, int ldw, void* out, int ldo, int M,
-                                  int N, int K, int epilogue, cudaStream_t stream) {
+                                  int N, int K, int epilogue, float limit, float slope, float shift,
+                                  cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || ldx < K || ldw < K || ldo < N) return RLLM_E_BADARG;
   if (K % 8 || ldx % 8 || ldw % 8 || M > 16) return RLLM_E_UNSUPPORTED;   // 16-byte loads of rows
@@ -337,7 +344,8 @@ RLLM_EXPORT int rllm_gemm_small_m(const void* x, int ldx, const void* W, int ldw
   switch (epilogue) {
     case EPI_BF16: return dispatch_mt<EPI_BF16>(xp, ldx, wp, ldw, out, ldo, M, N, K, 0, stream);
     case EPI_F32: return dispatch_mt<EPI_F32>(xp, ldx, wp, ldw, out, ldo, M, N, K, 0, stream);
-    case EPI_SILU: return dispatch_mt<EPI_SILU>(xp, ldx, wp, ldw, out, ldo, M, N, K, N, stream);
+    case EPI_SILU:
+      return dispatch_mt<EPI_SILU>(xp, ldx, wp, ldw, out, ldo, M, N, K, N, stream, GateAct{limit, slope, shift});
   }
   return RLLM_E_BADARG;
 }
@@ -348,16 +356,20 @@ RLLM_EXPORT int rllm_gemm_small_m_parts(int N) { return (N + 15) / 16; }
 // h[M, N] (float32, in place) += x[M, K] . W[N, K]^T for M <= 16 rows.  parts_out
 // [rllm_gemm_small_m_parts(N), M] receives, part by part, the sums of squares of 16 new values of each
 // row; with w_next (weight [N] of the norm that reads h next, float32 or bfloat16), scaled [M, N] receives
-// bfloat16(h * w_next).
+// bfloat16(h * w_next); with alpha (float32 [1]) and shift ([N], of w_next's type) too, that norm is the dynamic tanh
+// and scaled its whole result, bfloat16(tanh(alpha h) w_next + shift).
 RLLM_EXPORT int rllm_gemm_small_m_residual(const void* x, int ldx, const void* W, int ldw, float* h, int ldh,
                                            float* parts_out, const void* w_next, int w_is_f32, void* scaled,
-                                           int lds, int M, int N, int K, cudaStream_t stream) {
+                                           int lds, const float* alpha, const void* shift, int M, int N, int K,
+                                           cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  if (K <= 0 || ldx < K || ldw < K || ldh < N || !parts_out || (scaled && (!w_next || lds < N))) return RLLM_E_BADARG;
+  if (K <= 0 || ldx < K || ldw < K || ldh < N || !parts_out || (scaled && (!w_next || lds < N)) || ((alpha != nullptr) != (shift != nullptr)))
+    return RLLM_E_BADARG;
   if (K % 8 || ldx % 8 || ldw % 8 || M > 16) return RLLM_E_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return RLLM_E_BADARG;
   NormSide ns = {};
   ns.parts_out = parts_out; ns.w_next = w_next; ns.w_is_f32 = w_is_f32; ns.scaled = (bf16*)scaled; ns.lds = lds;
+  ns.alpha = alpha; ns.shift = shift;
   if (M <= 8) return launch_small_m<1, EPI_RESID, false>((const bf16*)x, ldx, (const bf16*)W, ldw, h, ldh, M, N, K, 0, ns, stream);
   return launch_small_m<2, EPI_RESID, false>((const bf16*)x, ldx, (const bf16*)W, ldw, h, ldh, M, N, K, 0, ns, stream);
 }
@@ -366,14 +378,15 @@ RLLM_EXPORT int rllm_gemm_small_m_residual(const void* x, int ldx, const void* W
 // `scaled` output of rllm_gemm_small_m_residual and parts [P, M] its partial sums, so that out is the
 // product of the RMS-normalised h with W.  epilogue 0 (bfloat16 out) or 2 (SiLU-gate), as above.
 RLLM_EXPORT int rllm_gemm_small_m_rstd(const void* x, int ldx, const float* parts, int P, float eps, const void* W,
-                                       int ldw, void* out, int ldo, int M, int N, int K, int epilogue,
-                                       cudaStream_t stream) {
+                                       int ldw, void* out, int ldo, int M, int N, int K, int epilogue, float limit,
+                                       float slope, float shift, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || ldx < K || ldw < K || ldo < N || P <= 0 || !parts || !(eps > 0.f)) return RLLM_E_BADARG;
   if (K % 8 || ldx % 8 || ldw % 8 || M > 16) return RLLM_E_UNSUPPORTED;
   if (((uintptr_t)x | (uintptr_t)W) & 15) return RLLM_E_BADARG;
   NormSide ns = {};
   ns.parts = parts; ns.P = P; ns.eps = eps; ns.width = K;
+  ns.ga = GateAct{limit, slope, shift};
   const bf16* xp = (const bf16*)x;
   const bf16* wp = (const bf16*)W;
   if (M <= 8) {

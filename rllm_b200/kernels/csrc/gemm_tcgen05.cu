@@ -27,6 +27,7 @@
 // The reference computes these products with a library call
 // (crates/rllm-model/src/layers.rs:162-175).
 #include "tcgen05.cuh"
+#include <math.h>
 
 #define TG_BM 128
 #define TG_BK 64
@@ -48,7 +49,7 @@ template <int BN, int EPI>
 __global__ void __launch_bounds__(TG_THREADS)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w,
                     void* __restrict__ out, int ldo, int M, int N, int K, int up_offset, int tiles_m,
-                    int num_tiles, int* __restrict__ err) {
+                    int num_tiles, int* __restrict__ err, GateAct ga) {
   constexpr int STAGES = tg_stages<BN>();
   constexpr int NOUT = (EPI == TG_EPI_SILU) ? BN / 2 : BN;     // output columns of a tile
   extern __shared__ unsigned char tg_raw[];
@@ -158,8 +159,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
-            const float g = __uint_as_float(r[j]);
-            r[j] = __float_as_uint(__fdividef(g, 1.0f + __expf(-g)) * __uint_as_float(u[j]));
+            const float g = fminf(__uint_as_float(r[j]), ga.limit);
+            const float up = fminf(fmaxf(__uint_as_float(u[j]), -ga.limit), ga.limit);
+            r[j] = __float_as_uint(__fdividef(g, 1.0f + __expf(-ga.slope * g)) * (up + ga.shift));
           }
         } else {
           asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -239,7 +241,8 @@ static int tg_num_sms() {
 
 template <int BN, int EPI>
 static int tg_launch(const void* a, int lda, const void* w, int ldw, int w_rows, void* out, int ldo, int M, int N,
-                     int K, int up_offset, int* err, cudaStream_t stream) {
+                     int K, int up_offset, int* err, cudaStream_t stream,
+                     GateAct ga = GateAct{INFINITY, 1.f, 0.f}) {
   constexpr int NOUT = (EPI == TG_EPI_SILU) ? BN / 2 : BN;
   CUtensorMap ma, mw;
   int rc = tg_make_map(&ma, a, M, K, lda, TG_BM);
@@ -259,15 +262,17 @@ static int tg_launch(const void* a, int lda, const void* w, int ldw, int w_rows,
   const int num_sms = tg_num_sms();
   const int grid = (int)(num_tiles < num_sms ? num_tiles : num_sms);
   gemm_tcgen05_kernel<BN, EPI><<<grid, TG_THREADS, tg_smem_bytes<BN>(), stream>>>(ma, mw, out, ldo, M, N, K, up_offset,
-                                                                                  tiles_m, (int)num_tiles, err);
+                                                                                  tiles_m, (int)num_tiles, err, ga);
   RLLM_LAUNCH_CHECK();
   return 0;
 }
 
 // epilogue 0: out bfloat16 [M, N]; 1: out float32 [M, N]; 2: W = [gate rows (N); up rows (N)] stacked,
-// out bfloat16 [M, N] = silu(A . gate^T) * (A . up^T).  err: the engine's error word (bit 16: a wait ran out).
+// out bfloat16 [M, N] = silu(A . gate^T) * (A . up^T), with the gate's constants limit, slope, shift (GateAct).  err:
+// the engine's error word (bit 16: a wait ran out).
 RLLM_EXPORT int rllm_gemm_tcgen05(const void* a, int lda, const void* w, int ldw, void* out, int ldo, int M, int N,
-                                  int K, int epilogue, int* err, cudaStream_t stream) {
+                                  int K, int epilogue, float limit, float slope, float shift, int* err,
+                                  cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || lda < K || ldw < K || ldo < N || !err) return RLLM_E_BADARG;
   // TMA: 16-byte aligned bases and row strides
@@ -294,7 +299,8 @@ RLLM_EXPORT int rllm_gemm_tcgen05(const void* a, int lda, const void* w, int ldw
     case TG_EPI_BF16: TG_BY_WIDTH(TG_EPI_BF16);
     case TG_EPI_F32: TG_BY_WIDTH(TG_EPI_F32);
     case TG_EPI_SILU:
-      return tg_launch<256, TG_EPI_SILU>(a, lda, w, ldw, 2 * N, out, ldo, M, N, K, N, err, stream);
+      return tg_launch<256, TG_EPI_SILU>(a, lda, w, ldw, 2 * N, out, ldo, M, N, K, N, err, stream,
+                                         GateAct{limit, slope, shift});
   }
   return RLLM_E_BADARG;
 }

@@ -153,24 +153,29 @@ hs_write_kernel(float* xs, const TY* y, const TW* g, const float* m, const float
 }
 
 // the dynamic tanh alone, on a float32 row set:  out[r] = tanh(alpha (x[row(r)] + delta[row(r)])) * w + c
-template <typename TO, typename TW>
+template <typename TO, typename TW, int V>
 __global__ void __launch_bounds__(HS_THREADS)
 dyt_kernel(float* x, const TO* delta, const int* rows, const float* alpha, const TW* w, const TW* c, TO* out,
            int H, long long total, int writeback) {
   const float al = alpha[0];
   pdl_wait();
   pdl_launch();
-  const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  const long long idx = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (idx >= total) return;
   const long long r = idx / H;
   const int i = (int)(idx - r * H);
   const size_t at = (size_t)(rows ? (long long)rows[r] : r) * H + i;
-  float v = x[at];
+  HsVec<V> v = hs_ld<V>(x + at);
   if (delta) {
-    v += to_f32(delta[at]);
-    if (writeback) x[at] = v;
+    const HsVec<V> dl = hs_ld<V>(delta + at);
+#pragma unroll
+    for (int e = 0; e < V; ++e) v.v[e] += dl.v[e];
+    if (writeback) hs_st<V>(x + at, v);
   }
-  out[idx] = from_f32<TO>(fmaf(tanhf(al * v), to_f32(w[i]), to_f32(c[i])));
+  const HsVec<V> ww = hs_ld<V>(w + i), cc = hs_ld<V>(c + i);
+#pragma unroll
+  for (int e = 0; e < V; ++e) v.v[e] = fmaf(tanhf(al * v.v[e]), ww.v[e], cc.v[e]);
+  hs_st<V>(out + idx, v);
 }
 
 static inline unsigned hs_blocks(long long total) { return (unsigned)((total + HS_THREADS - 1) / HS_THREADS); }
@@ -235,9 +240,15 @@ RLLM_EXPORT int rllm_dyt(float* x, const void* delta, const int* rows, const flo
   const long long total = (long long)R * H;
   if (total <= 0) return 0;
   if (!alpha || !w || !c) return RLLM_E_BADARG;
-  RLLM_DISPATCH_DTYPE(out_dtype, TO, RLLM_DISPATCH_DTYPE(w_dtype, TW,
-    (rllm_launch_pdl(dyt_kernel<TO, TW>, dim3(hs_blocks(total)), dim3(HS_THREADS), (size_t)0, stream, x,
-                     (const TO*)delta, rows, alpha, (const TW*)w, (const TW*)c, (TO*)out, H, total, writeback))));
+  const bool v4 = H % 4 == 0 && hs_aligned(x) && hs_aligned(delta) && hs_aligned(w) && hs_aligned(c) && hs_aligned(out);
+  RLLM_DISPATCH_DTYPE(out_dtype, TO, RLLM_DISPATCH_DTYPE(w_dtype, TW, {
+    if (v4)
+      rllm_launch_pdl(dyt_kernel<TO, TW, 4>, dim3(hs_blocks(total / 4)), dim3(HS_THREADS), (size_t)0, stream, x,
+                      (const TO*)delta, rows, alpha, (const TW*)w, (const TW*)c, (TO*)out, H, total, writeback);
+    else
+      rllm_launch_pdl(dyt_kernel<TO, TW, 1>, dim3(hs_blocks(total)), dim3(HS_THREADS), (size_t)0, stream, x,
+                      (const TO*)delta, rows, alpha, (const TW*)w, (const TW*)c, (TO*)out, H, total, writeback);
+  }));
   RLLM_LAUNCH_CHECK();
   return 0;
 }

@@ -133,14 +133,23 @@ def rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, token_seq: torch.T
            "rope_kv_write")
 
 
-def silu_mul(gate_up: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t, i] = silu(gate_up[t, i]) * gate_up[t, I + i]."""
+PLAIN_GATE = (float("inf"), 1.0, 0.0)
+
+
+def _gate_args(gate):
+    """(limit, slope, shift) of a gated product: g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = u kept
+    within +-limit; ``PLAIN_GATE`` is silu(g) u."""
+    return tuple(c_float(float(v)) for v in gate)
+
+
+def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, gate=PLAIN_GATE) -> None:
+    """out[t, i] = silu(gate_up[t, i]) * gate_up[t, I + i] (``gate``: other constants, see ``_gate_args``)."""
     lib = build.load_library("elementwise")
     T, I = out.shape
     assert gate_up.shape == (T, 2 * I) and gate_up.dtype is out.dtype
     _contig(gate_up, "gate_up"); _contig(out, "out")
     _check(lib.rllm_silu_mul(_ptr(gate_up), _ptr(out), c_int(dtype_code(out.dtype)), c_int(T), c_int(I),
-                             _stream()), "silu_mul")
+                             *_gate_args(gate), _stream()), "silu_mul")
 
 
 def attention_simt(q: torch.Tensor, q_stride: int, out: torch.Tensor, kcache: torch.Tensor,
@@ -181,7 +190,8 @@ FUSED_M_MAX = 16      # up to here a step goes through the forms of it that carr
                       # library's products with norm and SiLU kernels between them
 
 
-def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: str = "store") -> None:
+def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: str = "store",
+                 gate=PLAIN_GATE) -> None:
     """out = x . w^T for M <= 16 rows of bfloat16, bound by one read of w.
     epilogue "store": out [M, N] bfloat16 or float32.  "silu_mul": w = [gate rows;
     up rows] stacked (2 N rows), out [M, N] bfloat16 = silu(x gate^T) * (x up^T)."""
@@ -199,16 +209,17 @@ def gemm_small_m(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: 
         code = 1 if out.dtype is torch.float32 else 0
         assert out.dtype in (torch.float32, torch.bfloat16)
     _check(lib.rllm_gemm_small_m(_ptr(x), c_int(x.stride(0)), _ptr(w), c_int(w.stride(0)), _ptr(out),
-                                 c_int(out.stride(0)), c_int(M), c_int(N), c_int(K), c_int(code), _stream()),
-           "gemm_small_m")
+                                 c_int(out.stride(0)), c_int(M), c_int(N), c_int(K), c_int(code), *_gate_args(gate),
+                                 _stream()), "gemm_small_m")
 
 
 def gemm_small_m_residual(x: torch.Tensor, w: torch.Tensor, h: torch.Tensor,
-                          w_next: Optional[torch.Tensor]):
+                          w_next: Optional[torch.Tensor], tanh_norm=None):
     """h += x . w^T (h float32, in place) for M <= 16 rows of bfloat16.  Returns
     (parts, scaled): parts float32 [P, M], whose sum over P is each row's new sum of
     squares; scaled = bfloat16(h * w_next) [M, N] if the weight ``w_next`` of the norm
-    that reads h next is given, else None."""
+    that reads h next is given, else None.  ``tanh_norm`` = (alpha float32 [1], weight, shift) instead of ``w_next``: that
+    norm is a dynamic tanh, and scaled = bfloat16(tanh(alpha h) weight + shift), its whole result."""
     lib = build.load_library("gemm_small_m")
     M, K = x.shape
     N = w.shape[0]
@@ -217,20 +228,24 @@ def gemm_small_m_residual(x: torch.Tensor, w: torch.Tensor, h: torch.Tensor,
     assert x.stride(1) == 1 and w.stride(1) == 1
     P = int(lib.rllm_gemm_small_m_parts(c_int(N)))
     parts = torch.empty((P, M), dtype=torch.float32, device=x.device)
-    scaled = None
+    scaled = alpha = shift = None
+    if tanh_norm is not None:
+        alpha, w_next, shift = tanh_norm
+        assert alpha.dtype is torch.float32 and shift.dtype is w_next.dtype and shift.numel() == N and shift.is_contiguous()
     if w_next is not None:
         assert w_next.numel() == N and w_next.is_contiguous() and w_next.dtype in (torch.float32, torch.bfloat16)
         scaled = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     _check(lib.rllm_gemm_small_m_residual(_ptr(x), c_int(x.stride(0)), _ptr(w), c_int(w.stride(0)), _ptr(h),
                                           c_int(h.stride(0)), _ptr(parts), _ptr(w_next),
                                           c_int(1 if w_next is not None and w_next.dtype is torch.float32 else 0),
-                                          _ptr(scaled), c_int(N), c_int(M), c_int(N), c_int(K), _stream()),
+                                          _ptr(scaled), c_int(N), _ptr(alpha), _ptr(shift), c_int(M), c_int(N), c_int(K),
+                                          _stream()),
            "gemm_small_m_residual")
     return parts, scaled
 
 
 def gemm_small_m_rstd(x: torch.Tensor, parts: torch.Tensor, eps: float, w: torch.Tensor, out: torch.Tensor,
-                      epilogue: str = "store") -> None:
+                      epilogue: str = "store", gate=PLAIN_GATE) -> None:
     """out = (x . w^T) with row m scaled by 1 / sqrt(sum(parts[:, m]) / K + eps): with
     x and parts from ``gemm_small_m_residual`` this is rmsnorm(h) . w^T.  Epilogues
     as in ``gemm_small_m`` (bfloat16 out)."""
@@ -247,7 +262,7 @@ def gemm_small_m_rstd(x: torch.Tensor, parts: torch.Tensor, eps: float, w: torch
     assert out.shape == (M, N)
     _check(lib.rllm_gemm_small_m_rstd(_ptr(x), c_int(x.stride(0)), _ptr(parts), c_int(parts.shape[0]), c_float(eps),
                                       _ptr(w), c_int(w.stride(0)), _ptr(out), c_int(out.stride(0)), c_int(M),
-                                      c_int(N), c_int(K), c_int(code), _stream()), "gemm_small_m_rstd")
+                                      c_int(N), c_int(K), c_int(code), *_gate_args(gate), _stream()), "gemm_small_m_rstd")
 
 
 _one_wave_tiles = {}
@@ -302,7 +317,8 @@ def check_gemm_errors(device: torch.device) -> None:
         raise KernelError("; ".join(what or [f"error word {code}"]) + "; the result of that product is undefined")
 
 
-def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: str = "store") -> None:
+def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: str = "store",
+                 gate=PLAIN_GATE) -> None:
     """out = x . w^T for bfloat16 on the tcgen05 tensor cores (TMA in, TMEM accumulators).
     epilogue "store": out [M, N] bfloat16 or float32.  "silu_mul": w = [gate rows;
     up rows] stacked (2 N rows), out [M, N] bfloat16 = silu(x gate^T) * (x up^T)."""
@@ -319,7 +335,7 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: 
         assert out.shape == (M, N) and out.dtype in (torch.float32, torch.bfloat16)
         code = 1 if out.dtype is torch.float32 else 0
     _check(lib.rllm_gemm_tcgen05(_ptr(x), c_int(x.stride(0)), _ptr(w), c_int(w.stride(0)), _ptr(out),
-                                 c_int(out.stride(0)), c_int(M), c_int(N), c_int(K), c_int(code),
+                                 c_int(out.stride(0)), c_int(M), c_int(N), c_int(K), c_int(code), *_gate_args(gate),
                                  _ptr(gemm_error_word(x.device)), _stream()), "gemm_tcgen05")
 
 
@@ -1253,16 +1269,22 @@ def attention_simt_kv(q: torch.Tensor, q_stride: int, out: torch.Tensor, kcache:
                       block_table: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor, nq: int, nkv: int,
                       window: int, scale: float, err: torch.Tensor, keep_first: int = 0, chunk: int = 0,
                       softcap: float = 0.0, sinks: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                      gate_per_head: bool = False, slopes: Optional[torch.Tensor] = None) -> None:
+                      gate_per_head: bool = False, slopes: Optional[torch.Tensor] = None,
+                      shared_keys: Optional[int] = None) -> None:
     """``attention_simt`` where keys [pages, nkv, page, dk] and values [pages, nkv, page, dv] have sizes of their
     own: q rows of nq * dk, out [T, nq * dv]; any dk, dv up to 256.  ``keep_first``: with a window, the first
     that many keys of a sequence stay visible; ``chunk``: only keys of the query's own chunk of positions are;
     ``softcap``: scores become softcap * tanh(score / softcap); ``sinks`` float32 [nq]: exp(sink) joins each
     head's softmax denominator; ``gate`` [T, nq] (``gate_per_head``) or [T, nq * dv], a view with the rows'
     stride: the result is multiplied by its sigmoid; ``slopes`` float32 [nq]: slopes[h] * (query position - key
-    position) is taken off every score."""
+    position) is taken off every score.  ``shared_keys`` = dv: all heads read one key row a token ([pages, 1, page, dk])
+    and a token's value row holds the kv heads' values side by side ([pages, 1, page, nkv * places], dv of each)."""
     lib = build.load_library("attention_simt")
     T, dk, dv = out.shape[0], kcache.shape[3], vcache.shape[3]
+    v_ld = 0
+    if shared_keys is not None:
+        assert kcache.shape[1] == vcache.shape[1] == 1 and dv % nkv == 0
+        v_ld, dv = dv // nkv, int(shared_keys)
     _contig(out, "out"); _contig(kcache, "kcache"); _contig(vcache, "vcache"); _contig(block_table, "block_table")
     assert kcache.dtype is q.dtype and vcache.dtype is q.dtype and out.dtype is q.dtype and out.shape[1] == nq * dv
     if sinks is not None:
@@ -1276,7 +1298,8 @@ def attention_simt_kv(q: torch.Tensor, q_stride: int, out: torch.Tensor, kcache:
                                       c_float(scale), c_int(keep_first), c_int(chunk), c_float(softcap), _ptr(sinks),
                                       _ptr(gate), c_int(gate.stride(0) if gate is not None else 0),
                                       c_int(0 if gate is None else (1 if gate_per_head else 2)), _ptr(slopes),
-                                      _ptr(err), _stream()), "attention_simt_kv")
+                                      c_int(0 if shared_keys is None else 1), c_int(v_ld), _ptr(err), _stream()),
+           "attention_simt_kv")
 
 
 def rms_mean2(a: torch.Tensor, b: torch.Tensor, wa: torch.Tensor, wb: torch.Tensor, eps: float) -> torch.Tensor:
@@ -1663,3 +1686,92 @@ def channel_delta_step(a: torch.Tensor, c: Optional[torch.Tensor], x: torch.Tens
         c_int(dv), c_float(unit_eps), c_float(float(d) ** -0.5), c_float(eps), c_int(1 if early else 0), _ptr(err),
         _stream()), "channel_delta_step")
     return out
+
+
+# ---------------------------------------------------------------------------
+# linear attention with a matrix state (linear_state.cu)
+# ---------------------------------------------------------------------------
+def linear_state_scan(a: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, num_seqs: int,
+                      eps: float, err: torch.Tensor, decay: Optional[torch.Tensor] = None,
+                      inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, k_scale: float = 1.0,
+                      f_bias: Optional[torch.Tensor] = None, lower: Optional[torch.Tensor] = None,
+                      norm: Optional[torch.Tensor] = None, gated: bool = False,
+                      positions: Optional[torch.Tensor] = None, max_q_len: int = 1, early: bool = False) -> torch.Tensor:
+    """S_t = diag(f_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t over this step's tokens of every sequence, from and into the
+    sequences' slots of ``state`` (float32 [slots, heads, d, dv]); returns every head's o over its root mean square
+    (``eps`` under the root), times ``norm`` (float32 [dv]) if given, times silu(g) if ``gated``: [T, heads * dv] in a's
+    dtype.  a [T, .]: a token's projections [q | k or f | v | (g)], heads * d, heads * d, heads * dv (and heads * dv)
+    columns.  With ``decay`` (float32 [heads]): f is that number; q and k are rotated by ``positions`` over their first
+    ``rotary_dim`` dimensions (``inv_freq`` float64 [rotary_dim / 2], dimension i with i + rotary_dim / 2), then k is
+    multiplied by ``k_scale``.  With ``f_bias`` and ``lower`` (float32 [heads * d]): q <- silu(q),
+    f = lower + (1 - lower) sigmoid(f + f_bias), k = 1 - f.  ``early``: the kernel launched directly ahead does not write
+    ``state``, so that it may be fetched while that one still runs."""
+    lib = build.load_library("linear_state")
+    heads, d, dv = state.shape[1:]
+    T = a.shape[0]
+    assert a.stride(1) == 1 and a.shape[1] >= heads * (2 * d + dv * (2 if gated else 1))
+    assert state.dtype is torch.float32 and (decay is None) != (f_bias is None) and (f_bias is None) == (lower is None)
+    _contig(state, "state")
+    for t, n in ((decay, heads), (f_bias, heads * d), (lower, heads * d), (norm, dv)):
+        assert t is None or (t.dtype is torch.float32 and t.numel() == n and t.is_contiguous())
+    if rotary_dim:
+        assert inv_freq is not None and inv_freq.dtype is torch.float64 and inv_freq.numel() == rotary_dim // 2
+        assert positions is not None and positions.dtype is torch.int32 and positions.numel() == T
+    stride = a.stride(0) if T > 1 else a.shape[1]
+    out = torch.empty((T, heads * dv), dtype=a.dtype, device=a.device)
+    raw = torch.empty((T, heads * dv), dtype=torch.float32, device=a.device) \
+        if int(lib.rllm_linear_state_needs_raw(c_int(d), c_int(dv))) else None
+    _check(lib.rllm_linear_state_walk(_ptr(a), c_int(stride), c_int(dtype_code(a.dtype)), _ptr(decay),
+                                      _ptr(inv_freq if rotary_dim else None), c_int(rotary_dim), c_float(k_scale),
+                                      _ptr(f_bias), _ptr(lower), _ptr(norm), c_float(eps), c_int(1 if gated else 0),
+                                      _ptr(positions), _ptr(state), _ptr(q_start), _ptr(slots), c_int(state.shape[0]),
+                                      c_int(num_seqs), c_int(T), c_int(heads), c_int(d), c_int(dv), _ptr(out), _ptr(raw),
+                                      c_int(1 if early else 0), _ptr(err), _stream()), "linear_state_walk")
+    return out
+
+
+# ---------------------------------------------------------------------------
+# attention whose heads' scores are mixed (talking_heads.cu)
+# ---------------------------------------------------------------------------
+def talking_prep(qkv: torch.Tensor, positions: torch.Tensor, token_seq: torch.Tensor, bias: torch.Tensor,
+                 talk: torch.Tensor, inv_freq: Optional[torch.Tensor], rotary_dim: int, block_table: torch.Tensor,
+                 kcache: torch.Tensor, vcache: torch.Tensor, nq: int, nkv: int, dk: int, dv: int, err: torch.Tensor,
+                 v_other: Optional[torch.Tensor] = None, other_bias: Optional[torch.Tensor] = None,
+                 lam: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """qkv [T, nq dk + nkv dk + nkv dv], ``bias`` float32 over such a row.  Returns the mixed queries q' [T, nq * dkp]:
+    q'_h = [sum over the heads g of kv head 0 of talk[h, g] q_g | ... of the last kv head | zeros] (q biased and rotated),
+    whose product with a token's key row is head h's mixture of all heads' scores.  The key row [k_0 | k_1 | ... | zeros]
+    goes to kcache [pages, 1, page, dkp], the values to vcache [pages, 1, page, nkv * places] (zeros behind each head's
+    dv).  ``v_other`` [T, nkv dv] (a column slice will do), ``other_bias`` float32 [nkv dv], ``lam`` float32 [1]:
+    v <- (1 - lam) v + lam (v_other + other_bias)."""
+    lib = build.load_library("talking_heads")
+    T, dkp, vrow = qkv.shape[0], kcache.shape[3], vcache.shape[3]
+    assert qkv.stride(1) == 1 and qkv.shape[1] >= nq * dk + nkv * (dk + dv) and vrow % nkv == 0
+    assert kcache.shape[1] == vcache.shape[1] == 1 and kcache.dtype is qkv.dtype and vcache.dtype is qkv.dtype
+    assert bias.dtype is torch.float32 and bias.numel() == nq * dk + nkv * (dk + dv) and bias.is_contiguous()
+    assert talk.dtype is torch.float32 and talk.shape == (nq, nq) and talk.is_contiguous()
+    _contig(kcache, "kcache"); _contig(vcache, "vcache"); _contig(block_table, "block_table")
+    if rotary_dim:
+        assert inv_freq is not None and inv_freq.dtype is torch.float64 and inv_freq.numel() == rotary_dim // 2
+    if v_other is not None:
+        assert v_other.shape == (T, nkv * dv) and v_other.dtype is qkv.dtype and v_other.stride(1) == 1
+        assert other_bias.dtype is torch.float32 and other_bias.numel() == nkv * dv and other_bias.is_contiguous()
+        assert lam.dtype is torch.float32 and lam.numel() == 1
+    q_out = torch.empty((T, nq * dkp), dtype=qkv.dtype, device=qkv.device)
+    _check(lib.rllm_talking_prep(
+        _ptr(qkv), c_int(qkv.stride(0) if T > 1 else qkv.shape[1]), c_int(dtype_code(qkv.dtype)), _ptr(positions),
+        _ptr(token_seq), _ptr(bias), _ptr(talk), _ptr(inv_freq if rotary_dim else None), c_int(rotary_dim), _ptr(v_other),
+        c_int(v_other.stride(0) if v_other is not None else 0), _ptr(other_bias if v_other is not None else None),
+        _ptr(lam if v_other is not None else None), _ptr(block_table), c_int(block_table.shape[1]), _ptr(kcache),
+        _ptr(vcache), c_int(kcache.shape[2]), c_int(kcache.shape[0]), c_int(T), c_int(nq), c_int(nkv), c_int(dk),
+        c_int(dv), c_int(dkp), c_int(vrow // nkv), _ptr(q_out), _ptr(err), _stream()), "talking_prep")
+    return q_out
+
+
+def softcap_rows(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x <- cap * tanh(x / cap) in place; x float32, contiguous."""
+    lib = build.load_library("elementwise")
+    assert x.dtype is torch.float32 and cap > 0
+    _contig(x, "x")
+    _check(lib.rllm_softcap(_ptr(x), c_longlong(x.numel()), c_float(cap), _stream()), "softcap_rows")
+    return x

@@ -41,7 +41,15 @@ mean square and multiplied by nothing; ``q_temp`` = (coef, every): the query at 
 off the scaled score of key j, with slope_h = 2^(-x (h + 1) / num_heads) for head h (a bias linear in the
 distance, steeper for the first heads); ``qk_norm_span`` "row" (with ``qk_norm``): one root mean square over
 all of a token's query heads together, and one over its key heads, with weights [num_heads * head_dim] and
-[num_kv_heads * head_dim] ("head", the default: per head).
+[num_kv_heads * head_dim] ("head", the default: per head); ``bias`` "qkv": q, k and v have biases, the output
+projection has none; ``head_mix`` True: talking heads, score_h <- sum_g talk[h, g] score_g over all query heads, ahead
+of the mask and the softmax ("talk", [num_heads, num_heads]); ``value_mix`` (with ``head_mix``) "source" or "mixed": a
+"mixed" layer's values become (1 - lam) v + lam v_source ("value_mix", one number), v_source the same token's values in
+the "source" layer ahead of it; the mixed values are what is cached.
+
+With ``head_mix`` the mixture is moved to the queries: a token's keys of all kv heads form one row that every head
+reads, q'_h = [sum over the heads g of kv head 0 of talk[h, g] q_g | ... | of the last kv head], and q'_h . row is the
+mixed score (``kernels/csrc/talking_heads.cu``); the pages keep that row and the values of all kv heads side by side.
 
 A position part that rotates pairs (2i, 2i + 1) is served by the same kernels, which rotate halves: the rows of
 W_q, W_k, their biases and norm weights are put into the part's ``half_order`` when they are loaded.
@@ -88,6 +96,13 @@ class PagedAttention(Mixer):
         self.dv = int(p.get("v_dim") or self.d)
         self.qk_eps = float(p["qk_norm"]) if p.get("qk_norm") is not None else None
         self.bias = bool(p.get("bias", False))
+        if p.get("bias", False) not in (False, True, "qkv"):
+            raise ValueError(f"bias {p['bias']!r}; known: False, True, 'qkv'")
+        self.out_bias = self.bias and p.get("bias") != "qkv"
+        self.head_mix = bool(p.get("head_mix", False))
+        self.value_mix = p.get("value_mix")
+        if self.value_mix not in (None, "source", "mixed"):
+            raise ValueError(f"value_mix {self.value_mix!r}; known: None, 'source', 'mixed'")
         self.softcap = float(p["softcap"]) if p.get("softcap") else 0.0
         self.chunk = int(p["chunk"]) if p.get("chunk") else 0
         self.keep_first = int(p.get("keep_first") or 0)
@@ -113,7 +128,13 @@ class PagedAttention(Mixer):
             raise ValueError("softcap, chunk and keep_first must not be negative")
         # what the kernels of the Llama's form do not have: these go through the pages
         self.masked = bool(self.softcap or self.chunk or self.keep_first or self.sinks or self.gate or
-                           self.q_temp or self.slope_exp is not None)
+                           self.q_temp or self.slope_exp is not None or self.head_mix)
+        if self.value_mix and not self.head_mix:
+            raise ValueError("value_mix goes with head_mix")
+        if self.head_mix and (not self.bias or self.shares_kv or self.qk_eps is not None or self.softcap or self.chunk or
+                              self.sinks or self.gate or self.q_temp or self.slope_exp is not None):
+            raise ValueError("head_mix goes with biases, keys of the run's own, a window and kept first keys, and with no "
+                             "other option")
         # the Llama's form: rotation fused with the write
         self.plain = self.dv == self.d and self.qk_eps is None and not self.bias and not self.masked
         # keys and values of two sizes: where the larger one is a size of the tensor-core kernels, the pages keep
@@ -128,11 +149,19 @@ class PagedAttention(Mixer):
             raise ValueError(f"num_heads {self.nq} must be a multiple of num_kv_heads {self.nkv}")
         if self.plain and (self.d % 16 or self.d > 256):
             raise ValueError(f"head_dim {self.d}: the attention kernels take multiples of 16 up to 256")
+        # talking heads: a key row of all kv heads in whole panels of 64, value heads in places of 64 or 128 where the
+        # tensor-core kernels take them
+        self.dkp = self.dvp = 0
+        if self.head_mix:
+            self.dp = 0
+            self.dkp = -(-self.nkv * self.d // 64) * 64
+            self.dvp = 64 if self.dv <= 64 else (128 if self.dv <= 128 else self.dv)
         if self.dv > 256:
             raise ValueError(f"v_dim {self.dv}: the attention kernels take value heads up to 256")
         names = dict(p.get("tensor_names") or ())
         want = ["k", "o", "q", "v"] + (["k_norm", "q_norm"] if self.qk_eps is not None and self.qk_weights else []) + \
-            (["q_bias", "k_bias", "v_bias", "o_bias"] if self.bias else []) + \
+            (["q_bias", "k_bias", "v_bias"] if self.bias else []) + (["o_bias"] if self.out_bias else []) + \
+            (["talk", "value_mix"] if self.head_mix else []) + \
             (["sink"] if self.sinks and not self.zero_sinks else []) + (["g"] if self.gate else [])
         if sorted(names) != sorted(want):
             raise ValueError(f"an attention spec names its weights: tensor_names with the keys {sorted(want)}")
@@ -145,13 +174,15 @@ class PagedAttention(Mixer):
             raise ValueError(f"the rotation is of heads of {self.position.head_dim}, the mixer's heads have {self.d}")
         if not self.plain and self.position.fused_rotary() is None:
             raise ValueError("attention through the pages takes a rotation that its kernel can apply, or none")
+        if self.head_mix and self.pairs:
+            raise ValueError("head_mix takes a rotation of halves, or none")
         if self.shares_kv and self.bias:
             raise ValueError("a run that reads another's keys and values takes no biases")
         if not self.qk_weights and self.qk_eps is None:
             raise ValueError("qk_norm_weights False goes with qk_norm")
         self.gate_width = 0 if not self.gate else (self.nq if self.gate == "head" else self.nq * self.dv)
         self.w_qn = self.w_kn = None
-        self.b_qkv = self.b_o = self.sink = self.slopes = None
+        self.b_qkv = self.b_o = self.sink = self.slopes = self.talk = self.lam = None
         self.w_qkv: Optional[torch.Tensor] = None
         self.w_o: Optional[torch.Tensor] = None
         self._first_given = False
@@ -162,7 +193,9 @@ class PagedAttention(Mixer):
         return tuple(p + self.names[k] for k in ("q", "k", "v", "o"))
 
     def ignored_tensors(self) -> List[str]:
-        return self.position.ignored_tensors()
+        # (the layer that others mix in has a factor of its own that nothing uses)
+        unused = [self.prefix + self.names["value_mix"]] if self.head_mix and self.value_mix != "mixed" else []
+        return self.position.ignored_tensors() + unused
 
     def tensor_specs(self) -> List[TensorSpec]:
         q, k, v, o = self._names()
@@ -180,8 +213,13 @@ class PagedAttention(Mixer):
                                         init=("one_plus_normal", 0.1)))
         if self.bias:
             for key, n in (("q_bias", self.nq * self.d), ("k_bias", self.nkv * self.d), ("v_bias", self.nkv * self.dv),
-                           ("o_bias", self.hidden)):
+                           ("o_bias", self.hidden))[:4 if self.out_bias else 3]:
                 specs.append(TensorSpec(self.prefix + self.names[key], (n,), role="vector", init=("normal", 0.1)))
+        if self.head_mix:
+            specs.append(TensorSpec(self.prefix + self.names["talk"], (self.nq, self.nq), role="vector",
+                                    init=("normal", self.nq ** -0.5)))
+        if self.value_mix == "mixed":
+            specs.append(TensorSpec(self.prefix + self.names["value_mix"], (), role="vector", init=("normal", 0.5)))
         if self.sinks and not self.zero_sinks:
             specs.append(TensorSpec(self.prefix + self.names["sink"], (self.nq,), role="vector", init=("normal", 1.0)))
         if self.gate:
@@ -226,7 +264,12 @@ class PagedAttention(Mixer):
             # biases and sinks enter float32 arithmetic: kept so, whatever the run's dtype
             self.b_qkv = torch.cat([tensors[self.prefix + self.names[key]].float()
                                     for key in ("q_bias", "k_bias", "v_bias")]).contiguous()
-            self.b_o = tensors[self.prefix + self.names["o_bias"]].float().contiguous()
+            if self.out_bias:
+                self.b_o = tensors[self.prefix + self.names["o_bias"]].float().contiguous()
+        if self.head_mix:
+            self.talk = tensors[self.prefix + self.names["talk"]].float().contiguous()
+            if self.value_mix == "mixed":
+                self.lam = tensors[self.prefix + self.names["value_mix"]].float().reshape(1).contiguous()
         if self.zero_sinks:
             self.sink = torch.zeros(self.nq, dtype=torch.float32, device=self.w_o.device)
         elif self.sinks:
@@ -245,6 +288,8 @@ class PagedAttention(Mixer):
                 tensors[self.prefix + self.names["k_norm"]].to(self.w_qn.dtype).contiguous()
 
     def cache_need(self):
+        if self.head_mix:
+            return KVPagesNeed(1, self.dkp, self.window, v_dim=self.nkv * self.dvp, keep_first=self.keep_first)
         if self.dp:
             return KVPagesNeed(self.nkv, self.dp, self.window, keep_first=self.keep_first, chunk=self.chunk or None)
         return KVPagesNeed(self.nkv, self.d, self.window, v_dim=None if self.dv == self.d else self.dv,
@@ -252,7 +297,26 @@ class PagedAttention(Mixer):
 
     # -- compute ----------------------------------------------------------
     def fused_residual(self, num_rows: int, dtype: torch.dtype) -> bool:
-        return self.plain and fused_residual_takes(num_rows, dtype, self.w_qkv, self.w_o)
+        # talking heads: the output product of a decode step can carry the residual add and the next norm
+        return (self.plain or self.head_mix) and fused_residual_takes(num_rows, dtype, self.w_qkv, self.w_o)
+
+    def _attend_mixed_heads(self, qkv: torch.Tensor, ctx: StepContext, cache: KVCacheView) -> torch.Tensor:
+        """Talking heads: one kernel mixes the queries and writes the token's key row and values into the pages; the
+        attention reads everything from there."""
+        table = ctx.block_tables[cache.group]
+        inv_freq, rd = self.position.fused_rotary(qkv.device)
+        at, width = (self.nq + self.nkv) * self.d, self.nkv * self.dv
+        other = other_bias = None
+        if self.value_mix == "source":
+            ctx.extras["value_source"] = (qkv[:, at:at + width], self.b_qkv[at:at + width])
+        elif self.value_mix == "mixed":
+            other, other_bias = ctx.extras["value_source"]
+        q = ops.talking_prep(qkv, ctx.positions, ctx.token_seq, self.b_qkv, self.talk, inv_freq, rd, table, cache.k, cache.v,
+                             self.nq, self.nkv, self.d, self.dv, ctx.err, v_other=other, other_bias=other_bias, lam=self.lam)
+        out = torch.empty((qkv.shape[0], self.nq * self.dv), dtype=qkv.dtype, device=qkv.device)
+        ops.attention_simt_kv(q, q.stride(0), out, cache.k, cache.v, table, ctx.positions, ctx.token_seq, self.nq, self.nkv,
+                              int(self.window or 0), self.scale, ctx.err, keep_first=self.keep_first, shared_keys=self.dv)
+        return out
 
     def _attend_from_pages(self, qkv: torch.Tensor, ctx: StepContext, cache: KVCacheView) -> torch.Tensor:
         """Heads with norms or values of their own size: one kernel normalises the queries in place and writes
@@ -340,6 +404,8 @@ class PagedAttention(Mixer):
     def attend(self, qkv: torch.Tensor, ctx: StepContext, cache: KVCacheView) -> torch.Tensor:
         """From the tokens' projections (q, k and v heads side by side) to the attention's output
         [T, nq * d], before the output projection: position encoding, cache write, attention."""
+        if self.head_mix:
+            return self._attend_mixed_heads(qkv, ctx, cache)
         if not self.plain:
             return self._attend_from_pages(qkv, ctx, cache)
         x = qkv

@@ -4,6 +4,7 @@
 (crates/rllm-model/src/layers.rs:677-699):
     h   = x + mixer(norm_0(x))
     out = h + ffn(norm_1(h))
+(the feed-forward may be absent: out = h).
 The residual stream h is float32 and every add into it is a float32 add.  The
 last add of a block is not done here: the block returns (h, pending) with
 out = h + pending, and whichever norm reads the stream next adds ``pending``
@@ -41,14 +42,28 @@ from .registry import register_part
 from .spec import PartSpec
 
 
+class UnusedPart(Part):
+    """A part that its block does not run: a file that carries its tensors is no error."""
+    graph_safe = True
+
+    def __init__(self, part: Part):
+        super().__init__(part.spec, part.prefix)
+        self.part = part
+
+    def ignored_tensors(self) -> List[str]:
+        return [t.name for t in self.part.tensor_specs()] + self.part.ignored_tensors()
+
+
 @register_part("block", "pre_norm")
 class PreNormBlock:
-    def __init__(self, mixer: Mixer, ffn: FeedForward, norms: List[Norm]):
+    def __init__(self, mixer: Mixer, ffn: Optional[FeedForward], norms: List[Norm]):
         if len(norms) != 2:
             raise ValueError("a pre_norm block has two norms: before the mixer and before the feed-forward")
         self.mixer, self.ffn, self.norms = mixer, ffn, norms
 
     def parts(self):
+        if self.ffn is None:
+            return [self.norms[0], self.mixer, UnusedPart(self.norms[1])]
         return [self.norms[0], self.mixer, self.norms[1], self.ffn]
 
     takes_next_norm = True
@@ -56,12 +71,13 @@ class PreNormBlock:
     def _fused(self, num_rows: int, ctx: StepContext) -> bool:
         import os
         return (all(getattr(p, "fused_residual", None) is not None and p.fused_residual(num_rows, ctx.act_dtype)
-                    for p in (self.mixer, self.ffn))
+                    for p in ((self.mixer,) if self.ffn is None else (self.mixer, self.ffn)))
                 and all(hasattr(n, "scaled_input") for n in self.norms)
                 and os.environ.get("RLLM_FUSED_NORM") != "0")
 
     def forward(self, h: torch.Tensor, pending, ctx: StepContext, cache, next_norm=None):
         """``next_norm``: the norm that reads the stream after this block, if the caller knows it."""
+        trace = ctx.extras.get("residual_trace")         # a list: the stream after every layer (a copy)
         if self._fused(h.shape[0], ctx):
             xn = self.norms[0].scaled_input(pending) if isinstance(pending, RowSumsq) else None
             if xn is None:
@@ -69,8 +85,13 @@ class PreNormBlock:
                     xn = self.norms[0].forward(h, ctx.act_dtype)
                 else:
                     xn = self.norms[0].add_forward(h, pending)
-            stats = self.mixer.forward(xn, ctx, cache, residual=(h, self.norms[1]))
-            stats = self.ffn.forward(self.norms[1].scaled_input(stats), residual=(h, next_norm))
+            if self.ffn is None:
+                stats = self.mixer.forward(xn, ctx, cache, residual=(h, next_norm))
+            else:
+                stats = self.mixer.forward(xn, ctx, cache, residual=(h, self.norms[1]))
+                stats = self.ffn.forward(self.norms[1].scaled_input(stats), residual=(h, next_norm))
+            if trace is not None:
+                trace.append(h.clone())
             return h, stats
         if not isinstance(pending, torch.Tensor):
             pending = None                      # h is complete (whatever a block ahead prepared beside it)
@@ -78,9 +99,14 @@ class PreNormBlock:
             xn = self.norms[0].forward(h, ctx.act_dtype)
         else:
             xn = self.norms[0].add_forward(h, pending)
-        a = self.mixer.forward(xn, ctx, cache)
-        xn = self.norms[1].add_forward(h, a)
-        return h, self.ffn.forward(xn)
+        y = self.mixer.forward(xn, ctx, cache)
+        if self.ffn is not None:
+            y = self.ffn.forward(self.norms[1].add_forward(h, y))
+        if trace is not None:
+            ops.residual_add(h, y)
+            trace.append(h.clone())
+            return h, None
+        return h, y
 
 
 @register_part("block", "parallel_residual")

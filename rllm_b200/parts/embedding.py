@@ -26,7 +26,8 @@ class TokenEmbedding(Part):
         self.vocab = int(spec["vocab_size"])
         self.hidden = int(spec["hidden_size"])
         self.name = str(spec["name"])
-        self.scale = float(spec.get().get("scale") or 1.0)
+        scale = spec.get().get("scale")
+        self.scale = 1.0 if scale is None else float(scale)
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> List[TensorSpec]:
@@ -44,7 +45,8 @@ class TokenEmbedding(Part):
 
 class OutputHead(Part):
     """params: vocab_size, hidden_size, name, tied_to (name of the embedding
-    table that stands in when the file lacks ``name``; None: ``name`` is required)."""
+    table that stands in when the file lacks ``name``; None: ``name`` is required), softcap
+    (optional: the logits become softcap * tanh(logits / softcap))."""
 
     def __init__(self, spec: PartSpec, prefix: str = ""):
         super().__init__(spec, prefix)
@@ -52,6 +54,7 @@ class OutputHead(Part):
         self.hidden = int(spec["hidden_size"])
         self.name = str(spec["name"])
         self.tied_to = spec.get().get("tied_to")
+        self.softcap = spec.get().get("softcap")
         self.weight: Optional[torch.Tensor] = None
 
     def tensor_specs(self) -> List[TensorSpec]:
@@ -61,4 +64,5 @@ class OutputHead(Part):
         self.weight = tensors[self.name] if self.name in tensors else tensors[self.tied_to]
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
-        return linear(x, self.weight, out_dtype=torch.float32)
+        logits = linear(x, self.weight, out_dtype=torch.float32)
+        return logits if self.softcap is None else ops.softcap_rows(logits, float(self.softcap))

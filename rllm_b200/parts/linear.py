@@ -36,7 +36,8 @@ def linear(x, weight: torch.Tensor, out_dtype: Optional[torch.dtype] = None, res
         h, norm = residual
         assert fused_residual_takes(x.shape[0], x.dtype, weight)
         w_next = getattr(norm, "weight", None) if norm is not None and hasattr(norm, "scaled_input") else None
-        parts, scaled = ops.gemm_small_m_residual(x, weight, h, w_next)
+        tanh_norm = norm.elementwise() if w_next is not None and hasattr(norm, "elementwise") else None
+        parts, scaled = ops.gemm_small_m_residual(x, weight, h, w_next, tanh_norm=tanh_norm)
         return RowSumsq(parts, scaled, w_next)
     assert x.dim() == 2 and weight.dim() == 2 and x.shape[1] == weight.shape[1], (x.shape, weight.shape)
     if not x.is_cuda:

@@ -7,7 +7,10 @@ product with up are computed in float32.
 in the place of the SiLU (one product over the stacked weights, then one kernel
 for the activation and the product with up).
 
-params: hidden_size, intermediate_size, activation ("silu" if absent),
+With the SiLU, ``limit``, ``slope`` and ``up_shift`` give the gate other constants: with g = min(gate(x), limit) and
+u = up(x) kept within +-limit, down(g sigmoid(slope g) (u + up_shift)) (absent: no limit, 1, 0).
+
+params: hidden_size, intermediate_size, activation ("silu" if absent), limit, slope, up_shift,
 tensor_names (the names of the three weights below the part's prefix, keys
 "gate", "up", "down").
 """
@@ -36,6 +39,14 @@ class GatedMLP(FeedForward):
         self.activation = str(spec.get().get("activation") or "silu")
         if self.activation not in ops.ACTIVATIONS:
             raise ValueError(f"activation {self.activation!r}; known: {sorted(ops.ACTIVATIONS)}")
+        p = spec.get()
+        self.gate = (float(p["limit"]) if p.get("limit") is not None else float("inf"),
+                     float(p["slope"]) if p.get("slope") is not None else 1.0,
+                     float(p["up_shift"]) if p.get("up_shift") is not None else 0.0)
+        if self.gate != ops.PLAIN_GATE and self.activation != "silu":
+            raise ValueError("limit, slope and up_shift go with the activation 'silu'")
+        if not self.gate[0] > 0:
+            raise ValueError("limit must be positive")
         names = dict(spec.get().get("tensor_names") or ())
         if sorted(names) != ["down", "gate", "up"]:
             raise ValueError("a gated_mlp spec names its weights: tensor_names with the keys gate, up, down")
@@ -66,16 +77,16 @@ class GatedMLP(FeedForward):
             ops.act_mul(linear(x, self.w_gate_up), act, self.activation)
         elif isinstance(x, ScaledRows):
             # the rows' 1 / rms is applied to gate and up before the SiLU
-            ops.gemm_small_m_rstd(x.x, x.parts, x.eps, self.w_gate_up, act, "silu_mul")
+            ops.gemm_small_m_rstd(x.x, x.parts, x.eps, self.w_gate_up, act, "silu_mul", gate=self.gate)
         elif ops.small_m_takes(x, self.w_gate_up):
             # few rows: one kernel streams [Wgate; Wup] once and applies silu(gate) * up to its accumulators
-            ops.gemm_small_m(x, self.w_gate_up, act, "silu_mul")
+            ops.gemm_small_m(x, self.w_gate_up, act, "silu_mul", gate=self.gate)
         elif ops.tcgen05_takes(x, self.w_gate_up, silu=True):
             # many rows: tensor-core tiles of 128 gate and 128 up features, silu(gate) * up in the epilogue
-            ops.gemm_tcgen05(x, self.w_gate_up, act, "silu_mul")
+            ops.gemm_tcgen05(x, self.w_gate_up, act, "silu_mul", gate=self.gate)
         else:
             gate_up = linear(x, self.w_gate_up)                   # [T, 2I]
-            ops.silu_mul(gate_up, act)
+            ops.silu_mul(gate_up, act, gate=self.gate)
         return linear(act, self.w_down, residual=residual)
 
 

@@ -95,6 +95,10 @@ class DynamicTanh(Norm):
         """(alpha float32 [1], weight, shift): what a kernel needs to apply this norm to a value it holds."""
         return self.alpha, self.weight, self.shift
 
+    def scaled_input(self, stats: RowSumsq) -> Optional[torch.Tensor]:
+        """The normalised stream itself, if ``stats`` was prepared for this norm: nothing is left for its reader."""
+        return stats.scaled if stats.scaled is not None and stats.scaled_by is self.weight else None
+
     def forward(self, x: torch.Tensor, act_dtype: torch.dtype) -> torch.Tensor:
         out = torch.empty(x.shape, dtype=act_dtype, device=x.device)
         ops.dyt(x, self.alpha, self.weight, self.shift, out)
