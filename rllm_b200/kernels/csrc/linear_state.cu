@@ -278,3 +278,42 @@ RLLM_EXPORT int rllm_linear_state_walk(const void* a, int stride, int dtype, con
   RLLM_LAUNCH_CHECK();
   return 0;
 }
+
+RLLM_EXPORT int rllm_linear_state_chunk() { return LSM_C; }
+RLLM_EXPORT int rllm_linear_state_mma_takes(int d, int dv) { return d > 0 && dv > 0 && d <= 128 && dv <= 128 ? 1 : 0; }
+
+// cosine and sine of every (token, pair) of a step: table [T, half] pairs of floats
+RLLM_EXPORT int rllm_rotation_table(const int* positions, const double* inv_freq, int T, int half, void* table,
+                                    cudaStream_t stream) {
+  if (T <= 0 || half <= 0) return 0;
+  const long long n = (long long)T * half;
+  return (int)rllm_launch_pdl(ls_rotation_table_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), (size_t)0, stream,
+                              positions, inv_freq, half, (float2*)table, n);
+}
+
+// The same over long portions of bfloat16 rows (linear_state_mma.cuh): chunks chunk0 .. chunk0 + max_chunks - 1 of every
+// sequence's portion (a call goes on where the slots' states are), work num_seqs * max_chunks * heads * d * dv floats, gsum num_seqs * max_chunks * heads * d floats (decays per channel),
+// table from rllm_rotation_table (fixed decays with rd > 0), indexed by the same tokens as a's rows.
+RLLM_EXPORT int rllm_linear_state_chunked(const void* a, int stride, const float* decay, const void* table, int rd,
+                                          float k_scale, const float* f_bias, const float* lower, const float* norm_w,
+                                          float eps, int gated, float* state, float* work, float* gsum, const int* q_start,
+                                          const int* slots, int num_slots, int num_seqs, int chunk0, int max_chunks, int heads,
+                                          int d, int dv, void* out, int* err, cudaStream_t stream) {
+  if (num_seqs <= 0) return 0;
+  if (heads <= 0 || d <= 0 || dv <= 0 || num_slots <= 0 || max_chunks <= 0 || chunk0 < 0 || !work || !state)
+    return RLLM_E_BADARG;
+  if ((f_bias != nullptr) != (lower != nullptr) || (!f_bias && !decay) || (f_bias && !gsum)) return RLLM_E_BADARG;
+  if (rd < 0 || rd > d || (rd & 1) || (rd > 0 && !table) || stride < heads * (2 * d + dv * (gated ? 2 : 1))) return RLLM_E_BADARG;
+  if (d > 128 || dv > 128 || (long long)num_seqs * max_chunks > 65535) return RLLM_E_UNSUPPORTED;
+  const LsArgs p{stride, heads, d, dv, decay, nullptr, rd, k_scale, f_bias, lower, norm_w, eps, gated, nullptr};
+#define LSM_GO(D_, DV_)                                                                                                      \
+  (f_bias ? lsm_launch<D_, DV_, true>((const bf16*)a, p, (const float2*)table, state, work, gsum, q_start, slots, num_slots,  \
+                                      num_seqs, chunk0, max_chunks, (bf16*)out, err, stream)                                         \
+          : lsm_launch<D_, DV_, false>((const bf16*)a, p, (const float2*)table, state, work, gsum, q_start, slots, num_slots, \
+                                       num_seqs, chunk0, max_chunks, (bf16*)out, err, stream))
+  const int rc = d <= 64 ? (dv <= 64 ? LSM_GO(64, 64) : LSM_GO(64, 128)) : (dv <= 64 ? LSM_GO(128, 64) : LSM_GO(128, 128));
+#undef LSM_GO
+  if (rc) return rc;
+  RLLM_LAUNCH_CHECK();
+  return 0;
+}

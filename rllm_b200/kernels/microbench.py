@@ -12,6 +12,7 @@
     python -m rllm_b200.kernels.microbench mlstm_scan --tokens 2048 --heads 8 --head-dim 128 --v-dim 256
     python -m rllm_b200.kernels.microbench channel_delta --tokens 2048 --heads 16 --head-dim 128 --v-dim 128
     python -m rllm_b200.kernels.microbench ssd_scan --tokens 2048 --heads 64 --head-dim 64 --state 128 --groups 1
+    python -m rllm_b200.kernels.microbench linear_state --variant retention --tokens 2048 --heads 16 --head-dim 128
     python -m rllm_b200.kernels.microbench streams --tokens 2048 --hidden 2048 --streams 4
 
 Sizes default to the Llama-3.2-1B shape (32 heads, 8 kv heads, head 64, hidden
@@ -282,6 +283,32 @@ def lightning_scan(args) -> None:
           f"of rows and state, {4.0 * T * heads * d * dv / us / 1e6:.2f} TFLOP/s float32")
 
 
+def linear_state(args) -> None:
+    """The matrix-state recurrence with fixed decays (--variant retention) or decays per channel (--variant hgrn2), its
+    norm and gate, over one prompt portion, or one token of ``--batch`` sequences."""
+    heads, d, dv, gated = args.heads, args.head_dim, args.v_dim or args.head_dim, args.variant != "hgrn2"
+    q_start, _, slots, S, per = _one_sequence(args.tokens, args.batch)
+    T = S * per
+    bufs = [torch.randn(T, heads * (2 * d + (2 if gated else 1) * dv), device=DEV).bfloat16() for _ in range(4)]
+    state = torch.zeros(S, heads, d, dv, device=DEV)
+    err = torch.zeros(1, dtype=torch.int32, device=DEV)
+    pos = torch.arange(T, dtype=torch.int32, device=DEV)
+    if gated:
+        kind = dict(decay=torch.linspace(0.9, 0.999, heads, device=DEV), gated=True, rotary_dim=d, k_scale=d ** -0.5,
+                    inv_freq=torch.tensor([1e4 ** (-2.0 * i / d) for i in range(d // 2)], dtype=torch.float64, device=DEV))
+    else:
+        kind = dict(f_bias=torch.randn(heads * d, device=DEV) + 2, lower=torch.rand(heads * d, device=DEV) * 0.9,
+                    norm=torch.ones(dv, device=DEV))
+
+    def run(i):
+        ops.linear_state_scan(bufs[i % 4], state, q_start, slots, S, 1e-5, err, positions=pos, max_q_len=per,
+                              num_decode=S if per == 1 else 0, **kind)
+    us = time_graph_us(run, args.iters) if per == 1 else time_us(run, args.iters)
+    moved = T * heads * (4 * d + (6 if gated else 4) * dv) + 8 * S * heads * d * dv
+    print(f"linear_state ({'retention' if gated else 'hgrn2'}) tokens {T} ({S} sequences) heads {heads} x {d} x {dv}: "
+          f"{us:.1f} us, {moved / us / 1e3:.0f} GB/s of rows and state, {4.0 * T * heads * d * dv / us / 1e6:.2f} TFLOP/s")
+
+
 def mlstm_scan(args) -> None:
     """The matrix memory's recurrence over one prompt portion, or one token of ``--batch`` sequences."""
     heads, d, dv = args.heads, args.head_dim, args.v_dim or args.head_dim
@@ -412,7 +439,8 @@ def main(argv=None) -> int:
     p = argparse.ArgumentParser(prog="python -m rllm_b200.kernels.microbench", description=__doc__.split("\n\n")[0])
     p.add_argument("kernel", choices=["attention_decode", "attention_prefill", "gemm_small_m", "gemm_tcgen05",
                                       "latent_attention", "routed_experts", "lightning_scan", "selective_scan",
-                                      "streams", "mlstm_scan", "channel_delta", "channel_delta_step", "ssd_scan"])
+                                      "streams", "mlstm_scan", "channel_delta", "channel_delta_step", "ssd_scan",
+                                      "linear_state"])
     p.add_argument("--batch", type=int, default=8)
     p.add_argument("--context", type=int, default=4096)
     p.add_argument("--tokens", type=int, default=2048)
@@ -441,8 +469,8 @@ def main(argv=None) -> int:
     p.add_argument("--streams", type=int, default=4, help="streams: residual streams")
     p.add_argument("--experts", type=int, default=32)
     p.add_argument("--top", type=int, default=4)
-    p.add_argument("--variant", choices=["plain", "residual", "rstd"], default="plain",
-                   help="gemm_small_m: which epilogue / operand form")
+    p.add_argument("--variant", choices=["plain", "residual", "rstd", "retention", "hgrn2"], default="plain",
+                   help="gemm_small_m: which epilogue / operand form; linear_state: which recurrence")
     p.add_argument("--only", choices=["qkv", "o_proj", "gate_up", "down"], default=None,
                    help="gemm_small_m, gemm_tcgen05: this projection alone")
     p.add_argument("--impl", choices=["mma", "tcgen05"], default="mma",
@@ -455,7 +483,7 @@ def main(argv=None) -> int:
      "gemm_small_m": gemm_small_m, "gemm_tcgen05": gemm_tcgen05, "latent_attention": latent_attention,
      "routed_experts": routed_experts, "lightning_scan": lightning_scan, "selective_scan": selective_scan,
      "streams": streams, "mlstm_scan": mlstm_scan, "channel_delta": channel_delta,
-     "channel_delta_step": channel_delta_step,
+     "channel_delta_step": channel_delta_step, "linear_state": linear_state,
      "ssd_scan": ssd_scan}[args.kernel](args)
     return 0
 

@@ -1691,12 +1691,28 @@ def channel_delta_step(a: torch.Tensor, c: Optional[torch.Tensor], x: torch.Tens
 # ---------------------------------------------------------------------------
 # linear attention with a matrix state (linear_state.cu)
 # ---------------------------------------------------------------------------
+LINEAR_STATE_CHUNKED_FROM = 24          # longest portion from which bfloat16 steps go in chunks on the tensor cores
+LINEAR_STATE_WORK_BYTES = 64 << 20
+
+
+def rotation_table(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
+    """float32 [T, pairs, 2]: cosine and sine of positions[t] * inv_freq[i]."""
+    lib = build.load_library("linear_state")
+    T, half = positions.numel(), inv_freq.numel()
+    assert positions.dtype is torch.int32 and inv_freq.dtype is torch.float64
+    table = torch.empty((T, half, 2), dtype=torch.float32, device=positions.device)
+    _check(lib.rllm_rotation_table(_ptr(positions), _ptr(inv_freq), c_int(T), c_int(half), _ptr(table), _stream()),
+           "rotation_table")
+    return table
+
+
 def linear_state_scan(a: torch.Tensor, state: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, num_seqs: int,
                       eps: float, err: torch.Tensor, decay: Optional[torch.Tensor] = None,
                       inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, k_scale: float = 1.0,
                       f_bias: Optional[torch.Tensor] = None, lower: Optional[torch.Tensor] = None,
                       norm: Optional[torch.Tensor] = None, gated: bool = False,
-                      positions: Optional[torch.Tensor] = None, max_q_len: int = 1, early: bool = False) -> torch.Tensor:
+                      positions: Optional[torch.Tensor] = None, max_q_len: int = 1, early: bool = False,
+                      num_decode: int = 0, tables: Optional[dict] = None) -> torch.Tensor:
     """S_t = diag(f_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t over this step's tokens of every sequence, from and into the
     sequences' slots of ``state`` (float32 [slots, heads, d, dv]); returns every head's o over its root mean square
     (``eps`` under the root), times ``norm`` (float32 [dv]) if given, times silu(g) if ``gated``: [T, heads * dv] in a's
@@ -1705,7 +1721,11 @@ def linear_state_scan(a: torch.Tensor, state: torch.Tensor, q_start: torch.Tenso
     ``rotary_dim`` dimensions (``inv_freq`` float64 [rotary_dim / 2], dimension i with i + rotary_dim / 2), then k is
     multiplied by ``k_scale``.  With ``f_bias`` and ``lower`` (float32 [heads * d]): q <- silu(q),
     f = lower + (1 - lower) sigmoid(f + f_bias), k = 1 - f.  ``early``: the kernel launched directly ahead does not write
-    ``state``, so that it may be fetched while that one still runs."""
+    ``state``, so that it may be fetched while that one still runs.  Portions of bfloat16 from
+    ``LINEAR_STATE_CHUNKED_FROM`` tokens on (the first ``num_decode`` sequences, of one token each, aside) go in chunks
+    of 64 side by side on the tensor cores (heads up to 128 x 128); the result differs by rounding only.  ``tables`` keeps
+    the rotation tables of a step for its other calls."""
+    import os
     lib = build.load_library("linear_state")
     heads, d, dv = state.shape[1:]
     T = a.shape[0]
@@ -1719,6 +1739,34 @@ def linear_state_scan(a: torch.Tensor, state: torch.Tensor, q_start: torch.Tenso
         assert positions is not None and positions.dtype is torch.int32 and positions.numel() == T
     stride = a.stride(0) if T > 1 else a.shape[1]
     out = torch.empty((T, heads * dv), dtype=a.dtype, device=a.device)
+    if a.dtype is torch.bfloat16 and max_q_len >= LINEAR_STATE_CHUNKED_FROM and \
+            int(lib.rllm_linear_state_mma_takes(c_int(d), c_int(dv))) and os.environ.get("RLLM_LINEAR_STATE") != "simt":
+        S = num_seqs - num_decode
+        chunk = int(lib.rllm_linear_state_chunk())
+        chunks, per = -(-max_q_len // chunk), S * heads * d * dv * 4
+        calls = max(1, -(-chunks * per // LINEAR_STATE_WORK_BYTES), -(-chunks * S // 65535))
+        seg = -(-chunks // min(calls, chunks))
+        if seg * S <= 65535:
+            if num_decode:
+                out[:num_decode] = linear_state_scan(a[:num_decode], state, q_start, slots, num_decode, eps, err, decay,
+                                                     inv_freq, rotary_dim, k_scale, f_bias, lower, norm, gated,
+                                                     None if positions is None else positions[:num_decode], 1, early)
+            table = None
+            if rotary_dim:
+                tables = {} if tables is None else tables
+                key = (inv_freq.data_ptr(), rotary_dim)
+                if key not in tables:
+                    tables[key] = rotation_table(positions, inv_freq)
+                table = tables[key]
+            work = torch.empty(seg * S * heads * d * (dv + 1), dtype=torch.float32, device=a.device)
+            gsum = work[seg * S * heads * d * dv:]
+            for chunk0 in range(0, chunks, seg):
+                _check(lib.rllm_linear_state_chunked(
+                    _ptr(a), c_int(stride), _ptr(decay), _ptr(table), c_int(rotary_dim), c_float(k_scale), _ptr(f_bias),
+                    _ptr(lower), _ptr(norm), c_float(eps), c_int(1 if gated else 0), _ptr(state), _ptr(work), _ptr(gsum),
+                    _ptr(q_start[num_decode:]), _ptr(slots[num_decode:]), c_int(state.shape[0]), c_int(S), c_int(chunk0),
+                    c_int(seg), c_int(heads), c_int(d), c_int(dv), _ptr(out), _ptr(err), _stream()), "linear_state_chunked")
+            return out
     raw = torch.empty((T, heads * dv), dtype=torch.float32, device=a.device) \
         if int(lib.rllm_linear_state_needs_raw(c_int(d), c_int(dv))) else None
     _check(lib.rllm_linear_state_walk(_ptr(a), c_int(stride), c_int(dtype_code(a.dtype)), _ptr(decay),

@@ -71,7 +71,8 @@ class LinearStateMixer(Mixer):
     def _scan(self, a: torch.Tensor, ctx: StepContext, **kind) -> torch.Tensor:
         """``kind``: the arguments of ``ops.linear_state_scan`` that this kind of recurrence needs."""
         return ops.linear_state_scan(a, kind.pop("state"), ctx.q_start, ctx.state_slots, ctx.num_seqs, self.eps, ctx.err,
-                                     positions=ctx.positions, max_q_len=ctx.max_q_len, early=True, **kind)
+                                     positions=ctx.positions, max_q_len=ctx.max_q_len, early=True,
+                                     num_decode=ctx.num_decode, tables=ctx.extras.setdefault("tables", {}), **kind)
 
     def recurrence(self, a: torch.Tensor, ctx: StepContext, state: torch.Tensor) -> torch.Tensor:
         """From the tokens' projections to the output product's input."""
