@@ -39,7 +39,7 @@ NVCC_FLAGS = [
 SOURCES = ["elementwise", "attention_simt", "attention_mma", "attention_tcgen05", "gemm_f32", "gemm_small_m", "gemm_tcgen05", "sampling", "weights_rng",
            "layer_glue", "mingru", "latent_attention", "latent_attention_mma", "moe",
            "hyper_streams", "mixer_glue", "lightning", "selective_scan", "layernorm", "mlstm",
-           "ssd", "channel_delta", "linear_state", "talking_heads"]
+           "ssd", "channel_delta", "linear_state", "talking_heads", "shared_key_attention"]
 
 _lock = threading.Lock()
 _loaded: Dict[str, ctypes.CDLL] = {}

@@ -13,6 +13,7 @@
     python -m rllm_b200.kernels.microbench channel_delta --tokens 2048 --heads 16 --head-dim 128 --v-dim 128
     python -m rllm_b200.kernels.microbench ssd_scan --tokens 2048 --heads 64 --head-dim 64 --state 128 --groups 1
     python -m rllm_b200.kernels.microbench linear_state --variant retention --tokens 2048 --heads 16 --head-dim 128
+    python -m rllm_b200.kernels.microbench shared_key_attention --tokens 8192 --heads 16 --kv-heads 4 --head-dim 128 --window 1024
     python -m rllm_b200.kernels.microbench streams --tokens 2048 --hidden 2048 --streams 4
 
 Sizes default to the Llama-3.2-1B shape (32 heads, 8 kv heads, head 64, hidden
@@ -309,6 +310,59 @@ def linear_state(args) -> None:
           f"{us:.1f} us, {moved / us / 1e3:.0f} GB/s of rows and state, {4.0 * T * heads * d * dv / us / 1e6:.2f} TFLOP/s")
 
 
+def shared_key_attention(args) -> None:
+    """Attention over shared key rows (mixed heads): a prompt of ``--tokens``, or (--tokens 1) one token of ``--batch``
+    sequences at ``--context``; a key row has all kv heads' keys.  TFLOP/s over the visible pairs: as issued (every head
+    against the whole row), and as the unmixed heads and their mixture would count."""
+    H, G, d, dv, page, W, keep = args.heads, args.kv_heads, args.head_dim, args.v_dim or args.head_dim, args.page, args.window, args.keep_first
+    decode = args.tokens == 1
+    S, n, ctx = (args.batch, 1, args.context) if decode else (1, args.tokens, args.tokens)
+    dkp, dvp = -(-G * d // 64) * 64, 64 if dv <= 64 else 128
+    pages = -(-ctx // page)
+    nb = 2 if decode else 1
+    kc = [torch.randn(S * pages, 1, page, dkp, device=DEV).bfloat16() for _ in range(nb)]
+    vc = [torch.randn(S * pages, 1, page, G * dvp, device=DEV).bfloat16() for _ in range(nb)]
+    table = torch.arange(S * pages, dtype=torch.int32, device=DEV).view(S, pages)
+    q = torch.randn(S * n, H * dkp, device=DEV).bfloat16()
+    out = torch.empty(S * n, H * dv, dtype=torch.bfloat16, device=DEV)
+    q_start = torch.arange(0, S * n + 1, n, dtype=torch.int32, device=DEV)
+    lens = torch.full((S,), ctx, dtype=torch.int32, device=DEV)
+    err = torch.zeros(1, dtype=torch.int32, device=DEV)
+
+    def run(i):
+        if decode or args.impl == "mma":
+            ops.shared_key_attention_mma(q, out, kc[i % nb], vc[i % nb], table, q_start, lens, S, n, H, G, dv, W, keep, d ** -0.5,
+                                         err, ctx)
+        else:
+            ops.shared_key_attention_tcgen05(q, out, kc[0], vc[0], table, q_start, lens, 0, S, S * n, H, G, dv, W, keep,
+                                             d ** -0.5, err)
+    us = time_graph_us(run, args.iters) if decode else time_us(run, args.iters)
+    assert int(err.item()) == 0
+    pairs = sum(min(p + 1, W + min(keep, max(0, p + 1 - W))) if W else p + 1 for p in range(ctx - n, ctx)) * S
+    head = f"shared_key_attention tokens {S * n} context {ctx} heads {H}/{G} x {d}/{dv} window {W}+{keep}: {us:.1f} us"
+    if decode:
+        print(f"{head}, {pairs * 2.0 * G * (d + dv) / us / 1e3:.0f} GB/s of visible keys and values")
+    else:
+        print(f"{head}, {2e-6 * pairs * H * (dkp + dv) / us:.0f} TFLOP/s issued, {2e-6 * pairs * H * (d + H + dv) / us:.0f} unmixed")
+
+
+def talking_prep(args) -> None:
+    """The mixed queries, key rows and values of ``--tokens`` tokens."""
+    H, G, d, dv, page, T = args.heads, args.kv_heads, args.head_dim, args.v_dim or args.head_dim, args.page, args.tokens
+    dkp, dvp = -(-G * d // 64) * 64, 64 if dv <= 64 else 128
+    pages = -(-T // page)
+    kc, vc = (torch.zeros(pages, 1, page, w, device=DEV, dtype=torch.bfloat16) for w in (dkp, G * dvp))
+    width = H * d + G * (d + dv)
+    bufs = [torch.randn(T, width, device=DEV).bfloat16() for _ in range(4)]
+    inv = torch.tensor([1e4 ** (-2.0 * i / d) for i in range(d // 2)], dtype=torch.float64, device=DEV)
+    pos, err = torch.arange(T, dtype=torch.int32, device=DEV), torch.zeros(1, dtype=torch.int32, device=DEV)
+    seq, table = torch.zeros(T, dtype=torch.int32, device=DEV), torch.arange(pages, dtype=torch.int32, device=DEV).view(1, -1)
+    bias, talk = torch.randn(width, device=DEV), torch.randn(H, H, device=DEV)
+    us = time_us(lambda i: ops.talking_prep(bufs[i % 4], pos, seq, bias, talk, inv, d, table, kc, vc, H, G, d, dv, err), args.iters)
+    print(f"talking_prep tokens {T} heads {H}/{G} x {d}/{dv}: {us:.1f} us, "
+          f"{2.0 * T * (width + H * dkp + dkp + G * dvp) / us / 1e3:.0f} GB/s")
+
+
 def mlstm_scan(args) -> None:
     """The matrix memory's recurrence over one prompt portion, or one token of ``--batch`` sequences."""
     heads, d, dv = args.heads, args.head_dim, args.v_dim or args.head_dim
@@ -440,7 +494,7 @@ def main(argv=None) -> int:
     p.add_argument("kernel", choices=["attention_decode", "attention_prefill", "gemm_small_m", "gemm_tcgen05",
                                       "latent_attention", "routed_experts", "lightning_scan", "selective_scan",
                                       "streams", "mlstm_scan", "channel_delta", "channel_delta_step", "ssd_scan",
-                                      "linear_state"])
+                                      "linear_state", "shared_key_attention", "talking_prep"])
     p.add_argument("--batch", type=int, default=8)
     p.add_argument("--context", type=int, default=4096)
     p.add_argument("--tokens", type=int, default=2048)
@@ -484,6 +538,7 @@ def main(argv=None) -> int:
      "routed_experts": routed_experts, "lightning_scan": lightning_scan, "selective_scan": selective_scan,
      "streams": streams, "mlstm_scan": mlstm_scan, "channel_delta": channel_delta,
      "channel_delta_step": channel_delta_step, "linear_state": linear_state,
+     "shared_key_attention": shared_key_attention, "talking_prep": talking_prep,
      "ssd_scan": ssd_scan}[args.kernel](args)
     return 0
 

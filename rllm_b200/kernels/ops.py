@@ -1816,6 +1816,73 @@ def talking_prep(qkv: torch.Tensor, positions: torch.Tensor, token_seq: torch.Te
     return q_out
 
 
+def shared_key_tcgen05_takes(dtype: torch.dtype, nq: int, nkv: int, dkp: int, dvp: int, page_size: int) -> bool:
+    """Prompt portions go to the tcgen05 kernel when it takes the sizes (RLLM_ATTENTION=mma or simt keeps them off it)."""
+    import os
+    return (dtype is torch.bfloat16 and dkp % 64 == 0 and dkp <= 512 and dvp in (64, 128) and page_size in (16, 32, 64)
+            and nq // nkv <= 128 and os.environ.get("RLLM_ATTENTION") not in ("simt", "mma"))
+
+
+def shared_key_mma_takes(dtype: torch.dtype, nq: int, dkp: int, dvt: int) -> bool:
+    """bfloat16 sizes that the mma.sync kernel takes (RLLM_ATTENTION=simt keeps them on the CUDA cores)."""
+    import os
+    if dtype is not torch.bfloat16 or os.environ.get("RLLM_ATTENTION") == "simt":
+        return False
+    lib = build.load_library("shared_key_attention")
+    return bool(lib.rllm_shared_key_attention_mma_takes(c_int(nq), c_int(dkp), c_int(dvt)))
+
+
+def shared_key_attention_tcgen05(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
+                                 block_table: torch.Tensor, q_start: torch.Tensor, seq_lens: torch.Tensor, seq_begin: int,
+                                 seq_end: int, num_tokens: int, nq: int, nkv: int, dv: int, window: int, keep_first: int,
+                                 scale: float, err: torch.Tensor) -> None:
+    """Attention of the prompt portions of sequences seq_begin .. seq_end-1 where all heads read one key row a token: q
+    [T, nq * dkp], kcache [pages, 1, page, dkp], vcache [pages, 1, page, nkv * places] (dv of each), out [T, nq * dv];
+    key j is visible to position i if j <= i and (i - j < window (0: always) or j < keep_first)."""
+    lib = build.load_library("shared_key_attention")
+    _contig(q, "q"); _contig(out, "out"); _contig(kcache, "kcache"); _contig(vcache, "vcache"); _contig(block_table, "block_table")
+    dkp, dvp = kcache.shape[3], vcache.shape[3] // nkv
+    assert q.dtype is kcache.dtype is vcache.dtype is out.dtype is torch.bfloat16
+    assert q.shape[1] == nq * dkp and out.shape == (q.shape[0], nq * dv)
+    _check(lib.rllm_shared_key_attention_tcgen05(
+        _ptr(q), c_int(q.shape[0]), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_table), c_int(block_table.shape[1]),
+        _ptr(q_start), _ptr(seq_lens), c_int(seq_begin), c_int(seq_end), c_int(num_tokens), c_int(nq), c_int(nkv), c_int(dkp),
+        c_int(dv), c_int(dvp), c_int(kcache.shape[2]), c_int(kcache.shape[0]), c_int(window), c_int(keep_first),
+        c_float(scale), _ptr(err), _stream()), "shared_key_attention_tcgen05")
+
+
+def shared_key_attention_mma(q: torch.Tensor, out: torch.Tensor, kcache: torch.Tensor, vcache: torch.Tensor,
+                             block_table: torch.Tensor, q_start: torch.Tensor, seq_lens: torch.Tensor, num_seqs: int,
+                             max_q_len: int, nq: int, nkv: int, dv: int, window: int, keep_first: int, scale: float,
+                             err: torch.Tensor, max_seq_len: int) -> None:
+    """The same for sequences 0 .. num_seqs-1 on the mma.sync kernel; few rows: the keys in splits side by side.
+    ``max_seq_len`` bounds every length, ``max_q_len`` every portion."""
+    lib = build.load_library("shared_key_attention")
+    _contig(q, "q"); _contig(out, "out"); _contig(kcache, "kcache"); _contig(vcache, "vcache"); _contig(block_table, "block_table")
+    dkp, dvp = kcache.shape[3], vcache.shape[3] // nkv
+    assert q.dtype is kcache.dtype is vcache.dtype is out.dtype is torch.bfloat16
+    assert q.shape[1] == nq * dkp and out.shape == (q.shape[0], nq * dv)
+    rows = max_q_len * nq
+    tiles = num_seqs * -(-rows // (16 if rows <= 16 else 32))
+    keys = min(max_seq_len, window + max_q_len + keep_first) if window else max_seq_len
+    split, nsplit, work = 0, 1, None
+    if tiles <= 256 and keys > 128:
+        split = 64 if tiles <= 16 else (128 if tiles <= 48 else 256)
+        recent = -(-(window - 1 + max_q_len) // split) + 1 if window else -(-max_seq_len // split)
+        nsplit = min(-(-keep_first // split) + recent, -(-max_seq_len // split)) if window else recent
+        if 1 < nsplit <= 8192:
+            lib.rllm_shared_key_attention_mma_work.restype = c_longlong
+            n = int(lib.rllm_shared_key_attention_mma_work(c_int(num_seqs), c_int(max_q_len), c_int(nq), c_int(dvp), c_int(nsplit)))
+            work = torch.empty(n, dtype=torch.float32, device=q.device)
+        else:
+            split, nsplit = 0, 1
+    _check(lib.rllm_shared_key_attention_mma(
+        _ptr(q), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_table), c_int(block_table.shape[1]), _ptr(q_start),
+        _ptr(seq_lens), c_int(num_seqs), c_int(max_q_len), c_int(nq), c_int(nkv), c_int(dkp), c_int(dv), c_int(dvp),
+        c_int(kcache.shape[2]), c_int(kcache.shape[0]), c_int(window), c_int(keep_first), c_float(scale), c_int(split),
+        c_int(nsplit), _ptr(work), _ptr(err), _stream()), "shared_key_attention_mma")
+
+
 def softcap_rows(x: torch.Tensor, cap: float) -> torch.Tensor:
     """x <- cap * tanh(x / cap) in place; x float32, contiguous."""
     lib = build.load_library("elementwise")

@@ -314,8 +314,22 @@ class PagedAttention(Mixer):
         q = ops.talking_prep(qkv, ctx.positions, ctx.token_seq, self.b_qkv, self.talk, inv_freq, rd, table, cache.k, cache.v,
                              self.nq, self.nkv, self.d, self.dv, ctx.err, v_other=other, other_bias=other_bias, lam=self.lam)
         out = torch.empty((qkv.shape[0], self.nq * self.dv), dtype=qkv.dtype, device=qkv.device)
-        ops.attention_simt_kv(q, q.stride(0), out, cache.k, cache.v, table, ctx.positions, ctx.token_seq, self.nq, self.nkv,
-                              int(self.window or 0), self.scale, ctx.err, keep_first=self.keep_first, shared_keys=self.dv)
+        window, T, nd = int(self.window or 0), qkv.shape[0], ctx.num_decode
+        if self.scale <= 0 or not ops.shared_key_mma_takes(qkv.dtype, self.nq, self.dkp, self.nkv * self.dvp):
+            ops.attention_simt_kv(q, q.stride(0), out, cache.k, cache.v, table, ctx.positions, ctx.token_seq, self.nq,
+                                  self.nkv, window, self.scale, ctx.err, keep_first=self.keep_first, shared_keys=self.dv)
+            return out
+        heads, mask = (self.nq, self.nkv, self.dv), (window, self.keep_first, self.scale, ctx.err)
+        prompts = ops.shared_key_tcgen05_takes(qkv.dtype, self.nq, self.nkv, self.dkp, self.dvp, cache.k.shape[2])
+        if nd:
+            ops.shared_key_attention_mma(q, out, cache.k, cache.v, table, ctx.q_start, ctx.seq_lens, nd, 1, *heads, *mask,
+                                         max(ctx.seq_lens_host[:nd]))
+        if T > nd and prompts:
+            ops.shared_key_attention_tcgen05(q, out, cache.k, cache.v, table, ctx.q_start, ctx.seq_lens, nd, ctx.num_seqs,
+                                             T - nd, *heads, *mask)
+        elif T > nd:
+            ops.shared_key_attention_mma(q, out, cache.k, cache.v, table[nd:], ctx.q_start[nd:], ctx.seq_lens[nd:],
+                                         ctx.num_seqs - nd, ctx.max_q_len, *heads, *mask, ctx.max_seq_len)
         return out
 
     def _attend_from_pages(self, qkv: torch.Tensor, ctx: StepContext, cache: KVCacheView) -> torch.Tensor:
