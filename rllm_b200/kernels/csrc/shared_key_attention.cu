@@ -4,11 +4,12 @@
 // has moved to the queries (talking_heads.cu).
 //
 // The scheme is that of attention_tcgen05.cu: one CTA per (tile of 128 rows, kv head, sequence), a row a (token, head of
-// the kv head's group) pair; key tiles of 64 keys at absolute positions; S = Q K^T and P V as tcgen05.mma with
+// the kv head's group) pair; key tiles of 64 keys (128 with more
+// than four panels) at absolute positions; S = Q K^T and P V as tcgen05.mma with
 // accumulators in tensor memory; eight softmax warps, two threads a row; the kept first keys' tiles walked ahead of the
 // recent ones.  What differs: the contraction of S is up to eight panels long, so the keys come through a ring of single
-// panels (64 keys x 64 values), each handed back as soon as its four products are done; and several producer warps share
-// out a tile's pages (a box costs its warp some 140 cycles, and a tile has up to 8 panels x 4 pages of them).
+// panels (a tile's keys x 64 values), each handed back as soon as its four products are done; and several producer warps share
+// out a tile's pages (a box costs its warp some 140 cycles, and a tile has up to 8 panels x 8 pages of them).
 // Up to four panels two CTAs share an SM, with more one fills it.
 // Decoded tokens, and what the tcgen05 form does not take: the mma.sync kernel of latent_attention_mma.cuh, keys in splits
 // where there are few rows.
@@ -17,14 +18,14 @@
 #include "latent_attention_mma.cuh"
 
 #define SK_BM 128
-#define SK_BN 64
-#define SK_PANEL 8192            // bytes of a K or V panel: 64 keys x 64 values
 template <bool BIG> constexpr int sk_producers() { return BIG ? 4 : 2; }
 template <bool BIG> constexpr int sk_threads() { return 32 * (sk_producers<BIG>() + 9); }
-template <bool BIG> constexpr int sk_kstages() { return BIG ? 8 : 4; }
-template <int DV, bool BIG> constexpr int sk_vstages() { return BIG ? 2 : 128 / DV; }
+template <bool BIG> constexpr int sk_keys() { return BIG ? 128 : 64; }           // keys a tile
+template <bool BIG> constexpr int sk_panel() { return sk_keys<BIG>() * 128; }     // bytes of a K or V panel: a tile's keys x 64 values
+template <int DV, bool BIG> constexpr int sk_vstages() { return 128 / DV; }
+#define SK_KSTAGES 4
 template <int DV, bool BIG> constexpr int sk_smem(int panels) {
-  return panels * 16384 + sk_kstages<BIG>() * SK_PANEL + sk_vstages<DV, BIG>() * (DV / 64) * SK_PANEL + 512;
+  return panels * 16384 + SK_KSTAGES * sk_panel<BIG>() + sk_vstages<DV, BIG>() * (DV / 64) * sk_panel<BIG>() + 512;
 }
 
 template <int DV, bool BIG>
@@ -33,7 +34,8 @@ shared_key_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
                           const __grid_constant__ CUtensorMap map_v, bf16* out, const int* block_table, int max_blocks,
                           const int* q_start, const int* seq_lens, int seq_begin, int seq_end, int nq, int nkv, int panels,
                           int dv, int page_size, int num_pages, int window, int keep_first, float scale_log2, int* err) {
-  constexpr int NP = sk_producers<BIG>(), KST = sk_kstages<BIG>(), VST = sk_vstages<DV, BIG>(), DP = DV / 64;
+  constexpr int NP = sk_producers<BIG>(), KST = SK_KSTAGES, VST = sk_vstages<DV, BIG>(), DP = DV / 64;
+  constexpr int SK_BN = sk_keys<BIG>(), SK_PANEL = sk_panel<BIG>(), TMEM = BIG ? 512 : 256;
   constexpr int VSTAGE = DP * SK_PANEL;
   extern __shared__ __align__(1024) unsigned char sk_raw[];
   if (tg_smem(sk_raw) & 1023u) {                  // the swizzled tiles need 1024-byte alignment
@@ -41,8 +43,8 @@ shared_key_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
     return;
   }
   unsigned char* sQ = sk_raw;                     // panels x [128 rows][64 values], 128B swizzle
-  unsigned char* sK = sQ + panels * 16384;        // KST x [64 keys][64 values]
-  unsigned char* sV = sK + KST * SK_PANEL;        // VST x DP x [64 keys][64 values]
+  unsigned char* sK = sQ + panels * 16384;        // KST x [BN keys][64 values]
+  unsigned char* sV = sK + KST * SK_PANEL;        // VST x DP x [BN keys][64 values]
   unsigned long long* bars = (unsigned long long*)(sV + VST * VSTAGE);
   unsigned long long* q_full = bars;              // TMA -> MMA
   unsigned long long* k_full = bars + 1;          // [KST] TMA (all producers) -> MMA
@@ -99,14 +101,14 @@ shared_key_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
     asm volatile("prefetch.tensormap [%0];" ::"l"((unsigned long long)&map_v) : "memory");
   }
   if (warp == NP) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(tg_smem(tmem_slot)), "r"(256) : "memory");
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(tg_smem(tmem_slot)), "r"(TMEM) : "memory");
     asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
   }
   asm volatile("fence.proxy.async.shared::cta;" ::: "memory");   // the cleared ring, before TMA writes into it
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
   __syncthreads();
   asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-  const unsigned tmem_s = *tmem_slot, tmem_o = tmem_s + SK_BN, tmem_p = tmem_o + DV;   // 64 + DV + 32 + 4 <= 256 columns
+  const unsigned tmem_s = *tmem_slot, tmem_o = tmem_s + SK_BN, tmem_p = tmem_o + DV;   // BN + DV + BN / 2 + 4 <= TMEM columns
 
   if (warp < NP) {
     // ---- producers: warp w brings pages w, w + NP, ... of every tile, lane l the l-th of them
@@ -226,7 +228,8 @@ shared_key_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
       if (!ok) break;
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       float sc[HC];
-      tmem_ld32(tmem_s + lane_sel + half * HC, (unsigned*)sc);
+#pragma unroll
+      for (int c0 = 0; c0 < HC; c0 += 32) tmem_ld32(tmem_s + lane_sel + half * HC + c0, (unsigned*)(sc + c0));
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
       __syncwarp();
@@ -295,7 +298,8 @@ shared_key_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
       }
-      tmem_st16(tmem_p + lane_sel + half * (HC / 2), pk);
+      if constexpr (HC == 64) tmem_st32(tmem_p + lane_sel + half * (HC / 2), pk);
+      else tmem_st16(tmem_p + lane_sel + half * (HC / 2), pk);
       // rows of V at and behind the last visible key were never written by this sequence: cleared ahead of P V
       if (it == ntiles - 1) {
         const int st = it % VST;
@@ -355,7 +359,7 @@ shared_key_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
   asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
   __syncthreads();
   if (warp == NP) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_s), "r"(256) : "memory");
+    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_s), "r"(TMEM) : "memory");
   }
 }
 

@@ -13,6 +13,16 @@
 #include "common.cuh"
 #include <math.h>
 
+#define TH_PER 8                 // query heads a kv head that the quick form of the mixture takes
+
+__device__ __forceinline__ void th_store4(float* p, float4 v) { *(float4*)p = v; }
+__device__ __forceinline__ void th_store4(bf16* p, float4 v) {
+  uint2 r;
+  *(__nv_bfloat162*)&r.x = __floats2bfloat162_rn(v.x, v.y);
+  *(__nv_bfloat162*)&r.y = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)p = r;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 talking_prep_kernel(const T* qkv, int stride, const int* positions, const int* token_seq, const float* bias,
@@ -84,6 +94,31 @@ talking_prep_kernel(const T* qkv, int stride, const int* positions, const int* t
   __syncthreads();
   const int per = nq / nkv;
   T* qo = q_out + (size_t)t * nq * dkp;
+  if (per <= TH_PER && (dk & 3) == 0) {
+    // four neighbouring places of a kv head's part for a share of the heads: its query heads' values stay in registers
+    const int quads = nkv * dk / 4, shares = max(1, (int)blockDim.x / quads);
+    for (int e = threadIdx.x; e < quads * shares; e += blockDim.x) {
+      const int share = e / quads, c = (e - share * quads) * 4, g = c / dk;
+      float4 q[TH_PER];
+#pragma unroll
+      for (int u = 0; u < TH_PER; ++u)
+        if (u < per) q[u] = *(const float4*)&qs[(g * per + u) * dk + c - g * dk];
+      for (int h = share; h < nq; h += shares) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int u = 0; u < TH_PER; ++u) {
+          if (u < per) {
+            const float w = tk[h * nq + g * per + u];
+            v.x = fmaf(w, q[u].x, v.x); v.y = fmaf(w, q[u].y, v.y); v.z = fmaf(w, q[u].z, v.z); v.w = fmaf(w, q[u].w, v.w);
+          }
+        }
+        th_store4(qo + h * dkp + c, v);
+      }
+    }
+    const int pad = dkp - nkv * dk;
+    for (int e = threadIdx.x; e < nq * pad; e += blockDim.x) qo[e / pad * dkp + nkv * dk + e % pad] = from_f32<T>(0.f);
+    return;
+  }
   for (int e = threadIdx.x; e < nq * dkp; e += blockDim.x) {
     const int h = e / dkp, c = e - h * dkp, g = c / dk, i = c - g * dk;
     float v = 0.f;
@@ -109,6 +144,7 @@ RLLM_EXPORT int rllm_talking_prep(const void* qkv, int stride, int dtype, const 
     return RLLM_E_BADARG;
   const size_t smem = sizeof(float) * ((size_t)nq * dk + (size_t)nq * nq + rd);
   if (smem > 200 * 1024) return RLLM_E_UNSUPPORTED;
+  if (dkp % 4 || (((uintptr_t)q_out) & 15)) return RLLM_E_BADARG;
   RLLM_DISPATCH_DTYPE(dtype, TT, {
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(talking_prep_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
