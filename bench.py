@@ -540,6 +540,30 @@ BIRANEX_SIZES = {
 }
 
 
+def bikovik(layers, width, sheads, sdim, svdim, heads, kv_heads, dim, window, keep, ff, vocab):
+    """layers of the pattern [hgrn2, attention, retention, attention], each with a clamped dense feed-forward."""
+    rot = {"base": 500000.0, "dims": dim // 2}
+    state = {"heads": sheads, "dim": sdim, "vdim": svdim}
+    att = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "rot": rot, "v_mix": True,
+           "mask": {"size": window, "keep_first": keep}}
+    ret = dict(state, decay=[1.0 - 2.0 ** -(5 + 4.0 * h / sheads) for h in range(sheads)], rot={"base": 10000.0, "dims": sdim})
+    kinds = [("hgrn2", state), ("attention", att), ("retention", ret), ("attention", att)]
+    return {"architecture": "Bikovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 2.0},
+            "logit_softcap": 20.0, "max_positions": 8192,
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+                       for i in range(layers)]}
+
+
+# Bikovik beside Biranex (the closest dense design: layers with a matrix state, and windowed attention) of equal width,
+# layers, vocabulary, attention and matrix-state sizes, and the Llama of that width.
+BIKOVIK_SIZES = {
+    "w1024": dict(layers=4, width=1024, sheads=8, sdim=64, svdim=128, heads=16, kv_heads=4, dim=64, window=512, keep=4,
+                  ff=2048, vocab=32768),
+    "w2048": dict(layers=4, width=2048, sheads=16, sdim=128, svdim=128, heads=16, kv_heads=4, dim=128, window=1024, keep=4,
+                  ff=4096, vocab=32768),
+}
+
+
 def compare_designs(args):
     """Prefill and decode throughput of Fasulix at sizes that resemble a real model's layers (random weights)
     beside the Llama of equal size, through the same step function; and, from one eager prefill step and one
@@ -638,6 +662,23 @@ def compare_designs(args):
             # the convolutions' results, the decays' steps and beta in, o out (float32); the state in and out
             return 6.0 * a[0].shape[0] * heads * d * dv, 2.0 * a[0].numel() + 4.0 * (a[1].numel() + a[2].numel()) + \
                 4.0 * a[0].shape[0] * heads * dv + 8.0 * S * heads * d * dv
+        if name == "linear_state_scan":
+            heads, d, dv = a[1].shape[1:]
+            # a token's projections in, its results out; the state in and out
+            return 4.0 * a[0].shape[0] * heads * d * dv, 2.0 * a[0].numel() + 2.0 * a[0].shape[0] * heads * dv + \
+                8.0 * S * heads * d * dv
+        if name in ("shared_key_attention_tcgen05", "shared_key_attention_mma"):
+            nq, nkv, dv, window, keep = a[9:14] if name == "shared_key_attention_mma" else a[10:15]
+            dk = a[2].shape[3] // nkv
+            vis, keys = seen(window, keep, 0)
+            # the heads' scores, their mixture, the values: less than what is issued (every head against the whole row)
+            return 2.0 * (dk + nq + dv) * nq * vis, 2.0 * (keys * nkv * (dk + dv) + Tn * nq * (dk + dv))
+        if name == "talking_prep":
+            return 0.0, 2.0 * (a[0].numel() + Tn * (a[10] + 1) * a[8].shape[3] + Tn * a[9].shape[3])
+        if name == "dyt":
+            return 0.0, a[4].numel() * (8.0 if kw.get("delta") is None else 14.0)
+        if name == "softcap_rows":
+            return 0.0, 8.0 * a[0].numel()
         if name == "head_gated_rmsnorm":
             return 0.0, 8.0 * a[0].numel()
         if name in ("rms_mean2", "gated_rmsnorm"):
@@ -672,7 +713,8 @@ def compare_designs(args):
             "streams_read", "streams_write", "head_norm_kv_write", "attention_simt_kv", "rms_mean2", "gated_rmsnorm",
             "act_mul", "moe_choose_sigmoid", "weighted_slot_sum", "layernorm", "add_rows", "add_row_bias", "mlstm_scan",
             "head_gated_rmsnorm", "act", "sigmoid_gate", "postnorm_add", "ssd_scan", "silu_gated_group_rmsnorm",
-            "channel_delta_scan", "channel_delta_step", "activation_rows")]
+            "channel_delta_scan", "channel_delta_step", "activation_rows", "linear_state_scan", "talking_prep", "dyt",
+            "shared_key_attention_tcgen05", "shared_key_attention_mma", "softcap_rows")]
         saved, log = {}, []
 
         def wrap(name, fn):
@@ -800,6 +842,9 @@ def compare_designs(args):
         if args.design == "biranex":
             row["biranex"] = measure("biranex", biranex(**BIRANEX_SIZES[name]))
             row["fevolorn"] = measure("fevolorn", fevolorn(**FEVOLORN_SIZES[name]))
+        elif args.design == "bikovik":
+            row["bikovik"] = measure("bikovik", bikovik(**BIKOVIK_SIZES[name]))
+            row["biranex"] = measure("biranex", biranex(**BIRANEX_SIZES[name]))
         elif args.design == "munupel":
             row["munupel"] = measure("munupel", munupel(**MUNUPEL_SIZES[name]))
         else:
@@ -832,7 +877,7 @@ def main():
     ap.add_argument("--no-standin", action="store_true", help="skip the library-operator stand-in")
     ap.add_argument("--settle-steps", type=int, default=SETTLE_STEPS,
                     help="untimed decode steps of a device-timed point before its warm-up steps (0 for a short capture under a profiler)")
-    ap.add_argument("--design", default=None, choices=["biranex", "fasulix", "fevolorn", "munupel", "tibelix"],
+    ap.add_argument("--design", default=None, choices=["bikovik", "biranex", "fasulix", "fevolorn", "munupel", "tibelix"],
                     help="instead of the default workload: this design beside the Llama of equal size (prefill and "
                          "decode throughput, kernels against their rooflines)")
     ap.add_argument("--design-size", default=None, help="only this entry of the design comparison's sizes")
