@@ -18,6 +18,7 @@ GATE_SLOPE = 1.702
 
 
 def read_model_dir(model_dir: str, round_to: Optional[torch.dtype] = None):
+    """``round_to``: the matrices are rounded to it (vectors and head mixtures of a 32-bit file keep their digits)."""
     from safetensors import safe_open
     with open(os.path.join(model_dir, "config.json")) as f:
         cfg = json.load(f)
@@ -25,7 +26,8 @@ def read_model_dir(model_dir: str, round_to: Optional[torch.dtype] = None):
     with safe_open(os.path.join(model_dir, "model.safetensors"), framework="pt") as f:
         for n in f.keys():
             t = f.get_tensor(n)
-            w[n] = (t.to(round_to) if round_to is not None and t.is_floating_point() else t).to(F64)
+            matrix = t.dim() == 2 and not n.endswith(".talk")
+            w[n] = (t.to(round_to) if round_to is not None and matrix else t).to(F64)
     return cfg, w
 
 

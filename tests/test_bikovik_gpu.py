@@ -1,6 +1,8 @@
 """Bikovik on the GPU against the plain implementation (tests/plain_bikovik.py): every mechanism's kernels alone, then
 whole models through trace replay in every way of cutting, keys at the window's edges, and greedy generation through
 the entry point."""
+import copy
+import json
 import math
 
 import numpy as np
@@ -9,6 +11,7 @@ import torch
 
 import plain_bikovik as pb
 import replay_util as ru
+from bikovik_util import BK_A, BK_B, BK_C, att, hgrn2, ret, sharpen, write_model
 
 pytestmark = pytest.mark.gpu
 
@@ -293,3 +296,383 @@ def test_decoding_in_splits_equals_one_walk(H, G, d, dv, window, keep, monkeypat
             p = torch.softmax(((q[s].double() @ data[s][0].double().t()) * scale).masked_fill(~seen, -math.inf), dim=-1)
             want = torch.stack([p[h] @ data[s][1][:, h // (H // G), :dv].double() for h in range(H)]).reshape(-1)
             assert rel(out[s], want) <= 2e-2, (S, s)
+
+
+# ---------------------------------------------------------------------------
+# norm, gate, cap
+# ---------------------------------------------------------------------------
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("H", [45, 72, 2048])
+def test_dynamic_tanh_completes_the_stream_and_normalises_it(dtype, H):
+    from rllm_b200.kernels import ops
+    g = torch.Generator().manual_seed(H)
+    x, delta = torch.randn(7, H, generator=g) * 3, (torch.randn(7, H, generator=g) * 2).to(DT[dtype])
+    w = {"n": 1 + 0.2 * torch.randn(H, generator=g), "n.b": torch.randn(H, generator=g), "n.alpha": torch.tensor([0.8])}
+    w64 = {k: v.double() for k, v in w.items()}
+    rows = [5, 0, 5]
+    for d in (None, delta):
+        full = x.double() + (d.double() if d is not None else 0)
+        for pick in (None, rows):
+            xd = x.cuda()
+            out = torch.empty(7 if pick is None else 3, H, dtype=DT[dtype], device="cuda")
+            ops.dyt(xd, w["n.alpha"].cuda(), w["n"].cuda(), w["n.b"].cuda(), out, delta=None if d is None else d.cuda(),
+                    rows=None if pick is None else i32(pick), writeback=d is not None and pick is None)
+            want = pb.dynamic_tanh(w64, "n", full)
+            assert rel(out, want if pick is None else want[pick]) <= (1e-6 if dtype == "float32" else 5e-3)
+            assert rel(xd, full if d is not None and pick is None else x.double()) <= 1e-6
+
+
+@pytest.mark.parametrize("M", [1, 3, 8, 16])
+@pytest.mark.parametrize("N,K", [(72, 40), (128, 192), (2048, 512)])
+def test_a_decode_product_adds_into_the_stream_and_makes_the_next_norm(M, N, K):
+    """The residual epilogue with a dynamic tanh: the new stream, and its whole norm in bfloat16."""
+    from rllm_b200.kernels import ops
+    g = torch.Generator().manual_seed(N + M)
+    x, w = torch.randn(M, K, generator=g).bfloat16(), (torch.randn(N, K, generator=g) * 0.1).bfloat16()
+    h = torch.randn(M, N, generator=g) * 2
+    p = {"n": (1 + 0.2 * torch.randn(N, generator=g)), "n.b": torch.randn(N, generator=g), "n.alpha": torch.tensor([0.7])}
+    for vec in (torch.float32, torch.bfloat16):
+        pv = {k: (v if k == "n.alpha" else v.to(vec)) for k, v in p.items()}
+        hd = h.cuda()
+        _, scaled = ops.gemm_small_m_residual(x.cuda(), w.cuda(), hd, None,
+                                              tanh_norm=(pv["n.alpha"].cuda(), pv["n"].cuda(), pv["n.b"].cuda()))
+        want = h.double() + x.double() @ w.double().t()
+        assert rel(hd, want) <= 1e-5
+        assert rel(scaled, pb.dynamic_tanh({k: v.double() for k, v in pv.items()}, "n", want)) <= 5e-3
+
+
+@pytest.mark.parametrize("rows", [1, 8, 16, 40, 300])
+@pytest.mark.parametrize("dtype,mode", [("float32", ""), ("bfloat16", ""), ("bfloat16", "tcgen05"), ("bfloat16", "library")])
+@pytest.mark.parametrize("limit", [0.4, 7.0])
+def test_clamped_gate_in_every_form_of_the_product(rows, dtype, mode, limit, monkeypatch):
+    """Gate pre-activations far above the limit, both signs of the other factor beyond it."""
+    from rllm_b200.parts.registry import build_part
+    from rllm_b200.parts.spec import PartSpec
+    monkeypatch.setenv("RLLM_GEMM", mode)
+    g = torch.Generator().manual_seed(rows)
+    H, F = 64, 136
+    w = {"m.gate": torch.randn(F, H, generator=g) * 0.6, "m.up": torch.randn(F, H, generator=g) * 0.6,
+         "m.down": torch.randn(H, F, generator=g) * 0.2}
+    w = {k: v.to(DT[dtype]) for k, v in w.items()}
+    x = torch.randn(rows, H, generator=g).to(DT[dtype])
+    part = build_part("feed_forward", PartSpec.of("gated_mlp", hidden_size=H, intermediate_size=F, limit=limit, slope=1.702,
+                                                  up_shift=1.0, tensor_names={"gate": "gate", "up": "up", "down": "down"}), prefix="m.")
+    part.load({k: v.cuda() for k, v in w.items()})
+    want = pb.clamped_ff({k: v.double() for k, v in w.items()}, "m.", x.double(), limit)
+    assert rel(part.forward(x.cuda()), want) <= (1e-5 if dtype == "float32" else 1.5e-2)
+
+
+@pytest.mark.parametrize("shape", [(3, 97), (8, 32768), (1, 1)])
+def test_logit_cap(shape):
+    from rllm_b200.kernels import ops
+    x = torch.randn(*shape, generator=torch.Generator().manual_seed(1)) * 40
+    x[0, 0] = 1e8
+    assert rel(ops.softcap_rows(x.cuda(), 20.0), pb.soft_cap(x.double(), 20.0)) <= 1e-6
+
+
+# ---------------------------------------------------------------------------
+# whole models
+# ---------------------------------------------------------------------------
+CFG = {"A": BK_A, "B": BK_B, "C": BK_C}
+
+
+@pytest.fixture(scope="module")
+def bk_dirs(tmp_path_factory):
+    return {n: write_model(str(tmp_path_factory.mktemp("bk_" + n)), CFG[n], 61 + i, sharpen) for i, n in enumerate("ABC")}
+
+
+def plain_rows(folder, dtype, reqs):
+    cfg, w = pb.read_model_dir(folder, round_to=torch.bfloat16 if dtype == "bfloat16" else None)
+    return {r: pb.forward(cfg, w, toks).numpy() for r, toks in reqs.items()}
+
+
+def compare(got, want, reqs, dtype, what):
+    """float32: every position's largest difference against the largest logit.  bfloat16: root mean square over the
+    vocabulary against the logits' own."""
+    errs = []
+    for r, toks in reqs.items():
+        have = np.stack([got[(r, p)] for p in range(len(toks))])
+        assert np.isfinite(have).all()
+        if dtype == "float32":
+            err = np.abs(have - want[r]).max(axis=1) / np.abs(want[r]).max()
+            assert err.max() <= 1e-4, (what, r, int(err.argmax()), float(err.max()))
+        else:
+            errs.append(np.sqrt(((have - want[r]) ** 2).mean(axis=1)) / np.sqrt((want[r] ** 2).mean()))
+    if dtype == "bfloat16":
+        e = np.concatenate(errs)
+        assert np.median(e) <= 0.03 and (e > 0.08).mean() <= 0.02 and e.max() <= 0.2, (what, np.median(e), e.max())
+
+
+def make_requests(vocab, lengths, seed):
+    rng = np.random.default_rng(seed)
+    return {f"r{i}": [int(t) for t in rng.integers(0, vocab, size=n)] for i, n in enumerate(lengths)}
+
+
+@pytest.mark.parametrize("tokens", [75, 1])
+@pytest.mark.parametrize("name", ["A", "B", "C"])
+def test_layers_match_the_plain_residual_after_every_layer(bk_dirs, name, tokens):
+    """A prompt in one step, and its last token decoded; in bfloat16 the decode path with its fused norms runs too."""
+    from rllm_b200.engine.loading import load_model
+    from rllm_b200.engine.replay import TraceSession
+    toks = make_requests(CFG[name]["vocab"], [75], seed=2)["r0"]
+    for dtype in ("float32", "bfloat16"):
+        cfg, w = pb.read_model_dir(bk_dirs[name], round_to=DT[dtype])
+        want = []
+        pb.forward(cfg, w, toks, want)
+        _, model = load_model(bk_dirs[name], dtype=dtype)
+        sess = TraceSession(model, 128, 16, 2)
+        sess.runner.capture_graphs = False
+        trace, orig = [], sess.runner.build_context
+
+        def with_trace(entries):
+            ctx, a, b = orig(entries)
+            ctx.extras["residual_trace"] = trace
+            return ctx, a, b
+
+        if tokens == 1:
+            sess.step({"step": 0, "entries": [{"id": "a", "tokens": toks[:-1], "want": []}], "end": []})
+        sess.runner.build_context = with_trace
+        sess.step({"step": 1, "entries": [{"id": "a", "tokens": toks[-tokens:], "want": []}], "end": ["a"]})
+        assert len(trace) == len(want) == len(CFG[name]["layers"])
+        for i, (g, x) in enumerate(zip(trace, want)):
+            err = (g.double().cpu() - x[-tokens:]).pow(2).mean().sqrt() / x.pow(2).mean().sqrt()
+            assert float(err) <= (2e-5 if dtype == "float32" else 4e-2), (dtype, i, float(err))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,page", [("A", 16), ("A", 4), ("B", 16), ("B", 8), ("B", 64), ("C", 16)])
+def test_every_way_of_cutting_gives_the_plain_logits(bk_dirs, name, page, dtype):
+    """Whole prompts, token by token from the first token on, portions down to two tokens, and mixed batches of up to
+    four live requests whose pages and state slots are given back and used again (the pool holds exactly the peak);
+    every position's logits are compared."""
+    V = CFG[name]["vocab"]
+    reqs = make_requests(V, [61, 1, 2, 17, 150, 33, 5], seed=7)
+    want = plain_rows(bk_dirs[name], dtype, reqs)
+    for what, tb in (("whole", ru.trace_whole(reqs)), ("one by one", ru.trace_tail_decode(reqs, tail=1000)),
+                     ("tail decoded", ru.trace_tail_decode(reqs, tail=45)),
+                     ("portions", ru.trace_portions(reqs, seed=1)),
+                     ("mixed", ru.trace_mixed(reqs, seed=2, live=4, tail=6)),
+                     ("mixed b", ru.trace_mixed(reqs, seed=3, live=3, tail=30))):
+        got = ru.run_trace(bk_dirs[name], dtype, tb, V, page_size=page, max_live=4)
+        compare(got, want, reqs, dtype, f"{name}/{dtype}/page {page}/{what}")
+
+
+@pytest.mark.parametrize("dtype,name", [("float32", "A"), ("bfloat16", "B"), ("bfloat16", "A")])
+def test_long_prompts_behind_portions_that_end_anywhere(bk_dirs, dtype, name):
+    """Prompts of several chunks, whole and behind a first portion that ends inside a chunk, beside a decoded token."""
+    V = CFG[name]["vocab"]
+    reqs = make_requests(V, [520, 300], seed=4)
+    want = plain_rows(bk_dirs[name], dtype, reqs)
+    tb = ru.TraceBuilder()
+    a, b = reqs["r0"], reqs["r1"]
+    tb.step([("r0", a[:37]), ("r1", b[:299])])
+    tb.step([("r0", a[37:518]), ("r1", b[299:])], end=["r1"])
+    tb.step([("r0", a[518:519])])
+    tb.step([("r0", a[519:])], end=["r0"])
+    compare(ru.run_trace(bk_dirs[name], dtype, tb, V), want, reqs, dtype, "long prompts")
+
+
+@pytest.mark.parametrize("dtype,name", [("float32", "A"), ("bfloat16", "B")])
+def test_long_decoding_over_many_pages_beside_a_later_request(bk_dirs, dtype, name):
+    """A prompt of 3 tokens, then 260 tokens one by one (pages of 8; the windows pass over decoded tokens, pages behind
+    them are given back, the kept ones stay), beside a second request that starts later."""
+    V = CFG[name]["vocab"]
+    reqs = make_requests(V, [263, 120], seed=9)
+    want = plain_rows(bk_dirs[name], dtype, reqs)
+    tb = ru.TraceBuilder()
+    a, b = reqs["r0"], reqs["r1"]
+    tb.step([("r0", a[:3])])
+    for i in range(3, 263):
+        entries = [("r0", a[i:i + 1])]
+        j = i - 60
+        if j == 0:
+            entries.append(("r1", b[:25]))
+        elif 0 < j < 96:
+            entries.append(("r1", b[24 + j:25 + j]))
+        tb.step(entries, end=(["r0"] if i == 262 else []) + (["r1"] if j == 95 else []))
+    got = ru.run_trace(bk_dirs[name], dtype, tb, V, page_size=8)
+    compare(got, want, reqs, dtype, "long decoding")
+
+
+@pytest.mark.parametrize("dtype,heads,kv,dim,vdim", [("float32", 4, 2, 32, 24), ("bfloat16", 4, 2, 64, 64),
+                                                     ("bfloat16", 2, 2, 24, 40), ("bfloat16", 4, 4, 128, 128)])
+@pytest.mark.parametrize("window,keep,page", [(37, 4, 16), (64, 17, 16), (5, 1, 8)])
+def test_a_key_at_the_edges_of_the_window_and_of_the_kept_ones(tmp_path, dtype, heads, kv, dim, vdim, window, keep, page):
+    """One token of the sequence is the only key that the last query matches: at the window's last place and one behind
+    it, at the last kept place and one behind it; in prompts, behind portions and with the last tokens decoded.  The
+    rotation's base is so large that it does not move the score."""
+    cfg = {"architecture": "Bikovik", "vocab": 64, "width": 64, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+           "logit_softcap": 1000.0, "layers": [att(heads, kv, dim, vdim, 1.0, window, keep, 1e30, 4, False)]}
+    hot = 5
+
+    def edit(w):
+        q, k = w["l0.mix.q"], w["l0.mix.k"]
+        w["embed"].mul_(0.05)
+        w["embed"][hot] = 0.0
+        w["embed"][hot, 0] = 3.0                       # the key
+        w["embed"][hot + 1] = 0.0
+        w["embed"][hot + 1, 1] = 3.0                   # the query that matches it
+        w["l0.norm1"].fill_(1.0)
+        w["l0.norm1.b"].fill_(0.0)
+        w["l0.norm1.alpha"].fill_(1.0)
+        u = torch.randn(dim, generator=torch.Generator().manual_seed(1))
+        u[:4] = 0.0                                    # nothing in the dimensions that rotate
+        q.mul_(0.1)
+        k.mul_(0.1)
+        k[:, 0] = (u / u.norm() * 3.5).repeat(kv)
+        q[:, 1] = (u / u.norm() * 3.5).repeat(heads)
+        for n in ("q.b", "k.b"):
+            w["l0.mix." + n].mul_(0.1)
+        w["l0.mix.talk"].copy_(torch.eye(heads) + 0.05 * torch.randn(heads, heads, generator=torch.Generator().manual_seed(2)))
+        w["l0.mix.v"].mul_(30.0)
+        w["l0.mix.o"].mul_(10.0)
+    folder = write_model(str(tmp_path), cfg, 8, edit)
+    pcfg, pw = pb.read_model_dir(folder, round_to=torch.bfloat16 if dtype == "bfloat16" else None)
+    rng = np.random.default_rng(3)
+    for end in (window + keep, 3 * page - 1, 3 * page, 130):   # the last token's place
+        if end < window + keep:
+            continue
+        last = {}
+        for place in (end - window + 1, end - window, keep - 1, keep):
+            toks = [int(t) for t in rng.integers(8, 64, size=end + 1)]
+            toks[place], toks[end] = hot, hot + 1
+            want = last[place] = pb.forward(pcfg, pw, toks).numpy()[-1]
+            reqs = {"r": toks}
+            for tb in (ru.trace_whole(reqs), ru.trace_tail_decode(reqs, tail=1), ru.trace_tail_decode(reqs, tail=window + 3),
+                       ru.trace_portions(reqs, seed=end)):
+                row = ru.run_trace(folder, dtype, tb, 64, page_size=page)[("r", end)]
+                err = np.sqrt(((row - want) ** 2).mean()) / np.sqrt((want ** 2).mean())
+                assert err <= (1e-4 if dtype == "float32" else 0.04), (end, place, float(err))
+        for seen, hidden in ((end - window + 1, end - window), (keep - 1, keep)):
+            a, b = last[seen], last[hidden]
+            if hidden >= keep or hidden == keep:       # (behind the window, and no kept token)
+                if end - hidden >= window:
+                    assert np.sqrt(((a - b) ** 2).mean()) > 0.1 * np.sqrt((a ** 2).mean()), "the key would not show"
+
+
+@pytest.mark.parametrize("what", ["talk", "value mix", "lower bound", "decay", "gate", "far key"])
+def test_what_random_weights_might_hide_changes_the_result(bk_dirs, tmp_path, what):
+    """Each of these changes the plain logits clearly, and the engine follows the change, in prompts and in decoding."""
+    cfg = copy.deepcopy(BK_A)
+
+    def edit(w):
+        sharpen(w)
+        if what == "talk":
+            w["l1.mix.talk"].copy_(w["l1.mix.talk"].t().contiguous() * -1.0)
+        elif what == "value mix":
+            w["l4.mix.vmix"].fill_(3.0)
+        elif what == "lower bound":
+            w["l0.mix.lower"].fill_(0.97)
+        elif what == "gate":
+            w["l2.mix.g"].mul_(-1.0)
+    if what == "decay":
+        cfg["layers"][2]["mixer"]["decay"] = [0.5, 0.9999]
+    elif what == "far key":
+        cfg["layers"][1]["mixer"]["mask"]["keep_first"] = 0
+    folder = write_model(str(tmp_path), cfg, 61, edit)
+    reqs = make_requests(211, [70], seed=1)
+    before, want = plain_rows(bk_dirs["A"], "float32", reqs)["r0"], plain_rows(folder, "float32", reqs)
+    diff = np.sqrt(((want["r0"] - before)[30:] ** 2).mean()) / np.sqrt((before ** 2).mean())
+    assert diff > 0.02, diff
+    for tb in (ru.trace_whole(reqs), ru.trace_tail_decode(reqs, tail=30), ru.trace_portions(reqs, seed=3)):
+        compare(ru.run_trace(folder, "float32", tb, 211), want, reqs, "float32", what)
+
+
+def test_bfloat16_rounding_does_not_gather_in_the_states(tmp_path):
+    """Slow decays over a long prompt, recurrences alone: a state that passed through bfloat16, or decays that lost their
+    last digits, would drift; the error at the end is no larger than at the start."""
+    cfg = {"architecture": "Bikovik", "vocab": 128, "width": 64, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+           "logit_softcap": 100.0, "layers": [hgrn2(2, 32, 48), ret(2, 32, 48, [0.999, 0.9999], 500.0, 32)]}
+
+    def edit(w):
+        sharpen(w)
+        w["l0.mix.f.b"].fill_(8.0)
+    folder = write_model(str(tmp_path), cfg, 5, edit)
+    reqs = make_requests(128, [900], seed=1)
+    want = plain_rows(folder, "bfloat16", reqs)["r0"]
+    for tb in (ru.trace_whole(reqs), ru.trace_tail_decode(reqs, tail=300)):
+        got = ru.run_trace(folder, "bfloat16", tb, 128)
+        err = np.array([np.sqrt(((got[("r0", p)] - want[p]) ** 2).mean()) for p in range(900)]) / np.sqrt((want ** 2).mean())
+        assert np.median(err[-100:]) <= 1.5 * np.median(err[100:200]) and err.max() <= 0.1, (np.median(err), err.max())
+
+
+def test_fork_copies_pages_and_state(bk_dirs):
+    """A request forked in the middle of a page goes on independently of its parent."""
+    V = BK_A["vocab"]
+    a = make_requests(V, [90, 90], seed=31)
+    reqs = {"p": a["r0"], "c": a["r0"][:45] + a["r1"][45:]}
+    want = plain_rows(bk_dirs["A"], "float32", reqs)
+    tb = ru.TraceBuilder()
+    tb.step([("p", reqs["p"][:45])])
+    tb.step([("c", reqs["c"][45:70]), ("p", reqs["p"][45:46])], fork=[("p", "c")])
+    for i in range(46, 90):
+        tb.step([("p", reqs["p"][i:i + 1])] + ([("c", reqs["c"][24 + i:25 + i])] if i < 66 else []),
+                end=(["c"] if i == 65 else []) + (["p"] if i == 89 else []))
+    got = ru.run_trace(bk_dirs["A"], "float32", tb, V, max_tokens=256)
+    for p in range(45):
+        got[("c", p)] = got[("p", p)]
+    compare(got, want, reqs, "float32", "fork")
+
+
+def test_the_runner_as_a_program_and_pools_no_larger_than_asked(bk_dirs):
+    """bin/trace_run as a child process with a pool of exactly the peak of live tokens and its four slots."""
+    V = BK_B["vocab"]
+    reqs = make_requests(V, [40, 70, 9, 64, 3, 20], seed=13)
+    want = plain_rows(bk_dirs["B"], "float32", reqs)
+    tb = ru.trace_mixed(reqs, seed=5, live=4, tail=4)
+    got = ru.run_trace(bk_dirs["B"], "float32", tb, V, page_size=16, subprocess_mode=True, max_live=None)
+    compare(got, want, reqs, "float32", "child process")
+
+
+def plain_greedy(cfg, w, prompt, n_new):
+    seq, out = list(prompt), []
+    for _ in range(n_new):
+        t = int(torch.argmax(pb.forward(cfg, w, seq)[-1]))
+        out.append(t)
+        seq.append(t)
+    return out
+
+
+@pytest.mark.parametrize("dtype,name", [("float32", "A"), ("float32", "C"), ("bfloat16", "B")])
+def test_greedy_generation_through_the_entry_point(bk_dirs, dtype, name):
+    """Nine requests through LLM.generate with the scheduler cutting prompts into portions of at most 16 tokens beside
+    decoding requests, CUDA graphs for the decode steps, more requests than sequences at a time.  float32: the plain
+    implementation's tokens.  bfloat16: its choice at (nearly) all places where that is clear."""
+    from rllm_b200 import LLM, SamplingParams
+    V = CFG[name]["vocab"]
+    rng = np.random.default_rng(17)
+    prompts = [[int(t) for t in rng.integers(0, V, size=int(n))] for n in (5, 41, 1, 23, 60, 2, 9, 30, 14)]
+    n_new = 12
+    llm = LLM(bk_dirs[name], dtype="fp32" if dtype == "float32" else "bf16", block_size=8, num_gpu_blocks=96,
+              max_num_seqs=4, max_num_batched_tokens=24, long_prefill_token_threshold=16, enable_prefix_caching=False)
+    assert llm.engine.runner.capture_graphs
+    outs = llm.generate(prompts, SamplingParams(temperature=0.0, max_tokens=n_new, ignore_eos=True))
+    cfg, w = pb.read_model_dir(bk_dirs[name], round_to=torch.bfloat16 if dtype == "bfloat16" else None)
+    clear = wrong = 0
+    for p, o in zip(prompts, outs):
+        got = o.outputs[0].token_ids
+        assert len(got) == n_new
+        if dtype == "float32":
+            assert got == plain_greedy(cfg, w, p, n_new)
+            continue
+        rows = pb.forward(cfg, w, list(p) + got[:-1])[len(p) - 1:]
+        for t, row in zip(got, rows):
+            top = torch.topk(row, 2).values
+            if float(top[0] - top[1]) > 6e-2 * float(row.abs().max()):
+                clear += 1
+                wrong += t != int(torch.argmax(row))
+    assert dtype == "float32" or (clear >= 20 and wrong <= 0.05 * clear), (clear, wrong)
+    assert any(g.graph is not None for g in llm.engine.runner.graphs.values())
+    llm.engine.cache.check()
+    assert llm.engine.cache.usage()["num_requests"] == 0
+
+
+def test_generation_from_the_command_line(bk_dirs, capsys):
+    """``rllm generate`` on token ids: the plain implementation's greedy tokens."""
+    from rllm_b200.cli import main
+    prompt = make_requests(BK_A["vocab"], [19], seed=8)["r0"]
+    assert main(["generate", bk_dirs["A"], "--prompt-ids", ",".join(map(str, prompt)), "--max-tokens", "6", "--temperature", "0",
+                 "--dtype", "fp32", "--ignore-eos", "--num-gpu-blocks", "32", "--json"]) == 0
+    got = json.loads([l for l in capsys.readouterr().out.splitlines() if l.startswith("{")][-1])["token_ids"]
+    cfg, w = pb.read_model_dir(bk_dirs["A"])
+    assert got == plain_greedy(cfg, w, prompt, 6)
