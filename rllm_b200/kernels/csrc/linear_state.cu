@@ -77,8 +77,10 @@ ls_walk_kernel(const T* a, LsArgs p, float* state, const int* q_start, const int
         const size_t at = (size_t)(tb + tt) * p.stride + i;
         const float l = p.lower[h * d + i], z = to_f32(ak[at]) + p.f_bias[h * d + i];
         qs[e] = ls_silu(to_f32(aq[at]));
-        fs[e] = fmaf(1.0f - l, ls_sigmoid(z), l);
-        ks[e] = (1.0f - l) * ls_sigmoid(-z);
+        float on, off;
+        ls_sigmoids(z, &on, &off);
+        fs[e] = fmaf(1.0f - l, on, l);
+        ks[e] = (1.0f - l) * off;
       }
     } else {
       const int half = p.rd >> 1, items = d - half;

@@ -19,6 +19,12 @@ struct LsArgs {
 };
 
 __device__ __forceinline__ float ls_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+// sigmoid(z) and sigmoid(-z) = 1 - sigmoid(z), each with its digits, from one exponential
+__device__ __forceinline__ void ls_sigmoids(float z, float* pos, float* neg) {
+  const float e = expf(-fabsf(z)), r = 1.0f / (1.0f + e), s = e * r;
+  *pos = z >= 0.f ? r : s;
+  *neg = z >= 0.f ? s : r;
+}
 __device__ __forceinline__ float ls_silu(float z) { return z / (1.0f + expf(-z)); }
 
 template <typename T>

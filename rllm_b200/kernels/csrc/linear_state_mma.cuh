@@ -94,19 +94,31 @@ __device__ __forceinline__ void lsm_put4(bf16* hi, bf16* lo, int col, int left, 
 
 // Decays per channel: four neighbouring channels of a token: key, log2 of the decay
 __device__ __forceinline__ void lsm_gate4(const bf16* f, const LsArgs& p, int h, int i, bool on, bool wide, float (&k)[4], float (&lf)[4]) {
-  float z[4];
+  float z[4], lo[4], bi[4];
   const int left = p.d - i;
   ltc_fetch4<true>(f, on, wide, left, z);
+  if (wide && left >= 4) {                     // (d is a multiple of four: the vectors' rows are 16-byte aligned)
+    const float4 a = *(const float4*)(p.lower + h * p.d + i), b = *(const float4*)(p.f_bias + h * p.d + i);
+    lo[0] = a.x; lo[1] = a.y; lo[2] = a.z; lo[3] = a.w;
+    bi[0] = b.x; bi[1] = b.y; bi[2] = b.z; bi[3] = b.w;
+  } else {
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      lo[x] = x < left ? p.lower[h * p.d + i + x] : 0.f;
+      bi[x] = x < left ? p.f_bias[h * p.d + i + x] : 0.f;
+    }
+  }
 #pragma unroll
   for (int x = 0; x < 4; ++x) {
     k[x] = 0.f;
     lf[x] = 0.f;
     if (on && x < left) {
-      const float l = p.lower[h * p.d + i + x], zz = z[x] + p.f_bias[h * p.d + i + x];
-      const float kk = (1.0f - l) * ls_sigmoid(-zz);
+      float sg, sn;
+      ls_sigmoids(z[x] + bi[x], &sg, &sn);
+      const float kk = (1.0f - lo[x]) * sn;
       // the decay's logarithm from 1 - k where k is small, so that decays close to one keep their digits; decays below
       // 2^-100 count as that
-      const float ln = kk < 0.5f ? log1pf(-kk) : logf(fmaf(1.0f - l, ls_sigmoid(zz), l));
+      const float ln = kk < 0.5f ? log1pf(-kk) : logf(fmaf(1.0f - lo[x], sg, lo[x]));
       k[x] = kk;
       lf[x] = fmaxf(ln * 1.4426950408889634f, -100.f);
     }
@@ -610,7 +622,8 @@ static int lsm_launch(const bf16* a, LsArgs p, const float2* table, float* state
     allowed = true;
   }
   // rows that start on 8-byte boundaries are fetched four values a load (the rotated pairs' partners too)
-  const int wide = p.stride % 4 == 0 && p.d % 4 == 0 && p.dv % 4 == 0 && p.rd % 8 == 0 && (((uintptr_t)a) & 7) == 0;
+  const int wide = p.stride % 4 == 0 && p.d % 4 == 0 && p.dv % 4 == 0 && p.rd % 8 == 0 && (((uintptr_t)a) & 7) == 0 &&
+                   (((uintptr_t)p.lower | (uintptr_t)p.f_bias) & 15) == 0;
   const dim3 grid(p.heads, num_seqs * max_chunks);
   rllm_launch_pdl(ls_mma_pass1_kernel<D, DV, GATE>, grid, dim3(256), s1, stream, a, p, table, wide, work, gsum, q_start,
                   chunk0, max_chunks);
