@@ -171,7 +171,7 @@ template <int D, int DV, bool GATE> struct LsmSmem1 {
 };
 
 template <int D, int DV, bool GATE>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, D <= 64 ? 4 : 2)
 ls_mma_pass1_kernel(const bf16* a, LsArgs p, const float2* table, int wide_, float* work, float* gsum, const int* q_start,
                     int chunk0, int max_chunks) {
   extern __shared__ __align__(16) unsigned char lsm_raw[];
@@ -350,7 +350,7 @@ __device__ __forceinline__ void lsm_decayed_a(uint32_t (&hi)[4], uint32_t (&lo)[
 }
 
 template <int D, int DV, bool GATE>
-__global__ void __launch_bounds__(LSM_T2)
+__global__ void __launch_bounds__(LSM_T2, D <= 64 ? 2 : 1)      // (two blocks' shared memory fits an SM where D is 64)
 ls_mma_pass2_kernel(const bf16* a, LsArgs p, const float2* table, int wide_, const float* work, const int* q_start,
                     int chunk0, int max_chunks, bf16* out) {
   extern __shared__ __align__(16) unsigned char lsm_raw[];
